@@ -95,6 +95,8 @@ def plan_groups(cache_specs: dict[int, KVCacheSpec | StateSpec]) -> tuple[list[C
             name = f"window{spec.window}" if spec.window else "full"
             if spec.planes != 2:
                 name += f"_x{spec.planes}"
+            if spec.keep_first:
+                name += f"_keep{spec.keep_first}"
             if any(g.name == name for g in groups.values()):
                 name = f"{name}_h{spec.kv_heads}d{spec.head_dim}"
             groups[spec] = CacheGroup(len(groups), name, spec, [])
@@ -102,22 +104,23 @@ def plan_groups(cache_specs: dict[int, KVCacheSpec | StateSpec]) -> tuple[list[C
     return list(groups.values()), states
 
 
-def window_pages(window: int, step_tokens: int, page_size: int) -> int:
-    return math.ceil((window + step_tokens) / page_size) + 1
+def window_pages(window: int, step_tokens: int, page_size: int, keep_first: int = 0) -> int:
+    return math.ceil((window + step_tokens) / page_size) + 1 + math.ceil(keep_first / page_size)
 
 
 def split_budget(
     groups: list[CacheGroup], budget_bytes: int, page_size: int, element_size: int, max_num_sequences: int, step_tokens: int
 ) -> None:
     """Pages per group from a byte budget: a windowed group gets every sequence's window
-    (capped at half the budget), the others share the rest by bytes per token
-    (python/instinct/mlx_engine.py:149-171)."""
+    (capped at half the budget, or at an equal share when there are more than two), the others share the
+    rest by bytes per token (python/instinct/mlx_engine.py:149-171)."""
     remaining = budget_bytes
+    most = budget_bytes // max(2, sum(1 for g in groups if g.spec.window))
     for group in groups:
         if group.spec.window:
             page_bytes = group.bytes_per_token(element_size) * page_size
-            pages = max_num_sequences * window_pages(group.spec.window, step_tokens, page_size)
-            pages = min(pages, max(1, budget_bytes // 2 // page_bytes))
+            pages = max_num_sequences * window_pages(group.spec.window, step_tokens, page_size, group.spec.keep_first)
+            pages = min(pages, max(1, most // page_bytes))
             group.capacity_pages = pages
             remaining -= pages * page_bytes
     full = [g for g in groups if not g.spec.window]
@@ -184,7 +187,7 @@ class PagedCache:
         h = host()
         self.manager = h.CacheManager(
             page_size,
-            [h.GroupSpec(g.name, g.capacity_pages, g.spec.window) for g in self.groups],
+            [h.GroupSpec(g.name, g.capacity_pages, g.spec.window, g.spec.keep_first) for g in self.groups],
             self.state_slots,
             step_tokens,
         )
@@ -244,6 +247,7 @@ class PagedCache:
             max_pages=self.max_pages_per_request,
             page_size=self.page_size,
             window=group.spec.window,
+            keep_first=group.spec.keep_first,
         )
 
     def device_bytes(self) -> int:

@@ -1,3 +1,4 @@
+from .dugalix_config import DugalixConfig
 from .gunedra_config import GunedraConfig
 from .lerorax_config import LeroraxConfig
 from .zetizen_config import ZetizenConfig
@@ -13,6 +14,7 @@ from .registry import (
 __all__ = [
     "Architecture",
     "ConfigError",
+    "DugalixConfig",
     "GunedraConfig",
     "LeroraxConfig",
     "ModelConfig",

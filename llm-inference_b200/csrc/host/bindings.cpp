@@ -52,13 +52,14 @@ PYBIND11_MODULE(b200_host, m) {
       .def("refcount", &PagePool::refcount);
 
   py::class_<GroupSpec>(m, "GroupSpec")
-      .def(py::init([](std::string name, int capacity_pages, int window) {
-             return GroupSpec{std::move(name), capacity_pages, window};
+      .def(py::init([](std::string name, int capacity_pages, int window, int keep_first) {
+             return GroupSpec{std::move(name), capacity_pages, window, keep_first};
            }),
-           py::arg("name"), py::arg("capacity_pages"), py::arg("window") = 0)
+           py::arg("name"), py::arg("capacity_pages"), py::arg("window") = 0, py::arg("keep_first") = 0)
       .def_readwrite("name", &GroupSpec::name)
       .def_readwrite("capacity_pages", &GroupSpec::capacity_pages)
-      .def_readwrite("window", &GroupSpec::window);
+      .def_readwrite("window", &GroupSpec::window)
+      .def_readwrite("keep_first", &GroupSpec::keep_first);
 
   py::class_<CacheManager>(m, "CacheManager")
       .def(py::init<int, std::vector<GroupSpec>, int, int>(), py::arg("page_size"), py::arg("groups"),

@@ -70,6 +70,8 @@ CacheManager::CacheManager(int page_size, std::vector<GroupSpec> groups, int sta
   std::set<std::string> names;
   for (const auto& group : groups_) {
     if (group.window < 0) throw CacheError("a window cannot be negative");
+    if (group.keep_first < 0 || (group.keep_first > 0 && !group.window))
+      throw CacheError("only a windowed group keeps first positions, and not a negative number of them");
     if (!names.insert(group.name).second) throw CacheError("duplicate cache group " + group.name);
     pools_.emplace_back(group.capacity_pages);
   }
@@ -82,8 +84,10 @@ int CacheManager::group_index(const std::string& name) const {
   throw CacheError("unknown cache group " + name);
 }
 
+int CacheManager::kept_pages(const GroupSpec& group) const { return ceil_div(group.keep_first, page_size_); }
+
 int CacheManager::window_pages(const GroupSpec& group) const {
-  return ceil_div(group.window + step_tokens_, page_size_) + 1;
+  return ceil_div(group.window + step_tokens_, page_size_) + 1 + kept_pages(group);
 }
 
 std::vector<int> CacheManager::needs(int total_tokens) const {
@@ -192,7 +196,7 @@ void CacheManager::advance(RequestId id, int length) {
     // The next position is `length`; it sees positions > length - window.
     const int first_live_position = std::max(0, length - window + 1);
     const int first_live = std::min(static_cast<int>(table.size()), first_live_position / page_size_);
-    for (int index = e.trimmed[g]; index < first_live; ++index) {
+    for (int index = std::max(e.trimmed[g], kept_pages(groups_[g])); index < first_live; ++index) {
       const int page = table[index];
       if (page < 0) continue;
       pools_[g].release(page);
@@ -261,7 +265,7 @@ CacheStats CacheManager::stats() const {
       std::int64_t held = 0;
       for (int page : e.tables[0]) held += page >= 0 ? page_size_ : 0;
       const int window = groups_[0].window;
-      const std::int64_t live = window ? std::min(e.length, window) : e.length;
+      const std::int64_t live = window ? std::min<std::int64_t>(e.length, static_cast<std::int64_t>(window) + groups_[0].keep_first) : e.length;
       out.internal_fragmentation_tokens += std::max<std::int64_t>(0, held - live);
     }
   }

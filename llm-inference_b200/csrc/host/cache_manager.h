@@ -57,6 +57,7 @@ struct GroupSpec {
   std::string name;
   int capacity_pages{0};
   int window{0};  // 0: every earlier position stays visible
+  int keep_first{0};  // with a window: the first this many positions stay visible too
 };
 
 struct GroupStats {
@@ -82,7 +83,8 @@ struct CacheStats {
 class CacheManager {
  public:
   // `step_tokens` bounds how many positions one request can add in one step; it sizes the
-  // reservation of windowed groups (window + step_tokens positions, plus one page of slack).
+  // reservation of windowed groups (window + step_tokens positions, plus one page of slack, plus the
+  // pages of the positions that stay visible from the start).
   CacheManager(int page_size, std::vector<GroupSpec> groups, int state_slots, int step_tokens);
 
   int page_size() const { return page_size_; }
@@ -106,7 +108,7 @@ class CacheManager {
   // Give the request a page for every position below `end`.
   void ensure(RequestId id, int end);
   // Positions below `length` now hold keys and values; windowed groups give back the pages
-  // that no position >= length can see.
+  // that no position >= length can see (the pages of the first `keep_first` positions stay).
   void advance(RequestId id, int length);
   // Give back every page, the unused reservation and the slot.
   void release(RequestId id);
@@ -137,6 +139,7 @@ class CacheManager {
     bool has_reservation{false};
   };
 
+  int kept_pages(const GroupSpec& group) const;
   int window_pages(const GroupSpec& group) const;
   int take_page(Entry& entry, int g);
   Entry& entry(RequestId id);

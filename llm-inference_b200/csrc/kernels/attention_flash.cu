@@ -19,8 +19,12 @@
 //     starts fetching keys that earlier steps wrote before it waits for the kernel in front
 //     of it on the stream, which only produces the newest key.
 // Masking follows python/instinct/batches.py:110-113: key <= query position, and with a
-// window key > position - window.
+// window key > position - window. Behind a window the first `keep_first` keys of a request may
+// stay visible (FORM_KEPT): the walk takes their tiles first, then the window's. FORM_SIGMOID turns
+// a score into a weight by a sigmoid instead of a softmax: no maximum, no sum, no rescaling.
 #include <cuda.h>
+
+#include <type_traits>
 
 #include "common.cuh"
 
@@ -55,6 +59,7 @@ struct FlashParams {
   int q_heads, kv_heads, group;
   int page_shift, page_mask;
   int window;
+  int keep_first;     // FORM_KEPT and FORM_SIGMOID: the first this many keys stay visible in front of the window
   int splits;
   int cluster_merge;  // the splits of a (request, kv head) are one thread-block cluster and merge on chip
   int value_head;     // >= 0: every query head's weights meet the values of this kv head instead of its own
@@ -120,6 +125,12 @@ __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) {
   return *reinterpret_cast<uint32_t*>(&v);
 }
 
+// What the kernel does to scores; one instantiation per form (see paged_flash_attention_kernel).
+enum : int { FORM_SOFTMAX = 0, FORM_SHAPED = 1, FORM_KEPT = 2, FORM_SIGMOID = 3 };
+
+// 1 / (1 + 2^-x) with the fast exponential and division; a masked score (-inf) weighs nothing.
+__device__ __forceinline__ float sigmoid_base2(float x) { return __fdividef(1.f, 1.f + exp2f(-x)); }
+
 // Byte offset of 16-byte chunk `chunk` of row `row` in a swizzled [rows][HEAD_DIM] bf16 tile.
 template <int HEAD_DIM>
 __device__ __forceinline__ int tile_offset(int row, int chunk) {
@@ -128,14 +139,35 @@ __device__ __forceinline__ int tile_offset(int row, int chunk) {
 
 // Copies keys and values [tile_start, tile_start + 64) of one kv head into their shared-memory
 // tiles; rows outside [lo, hi] are zero-filled (they may lie in pages the request no longer
-// holds). The block-table entries of all of a thread's rows are fetched first, in one batch
+// holds), except those of the first `keep` keys, whose pages a request never gives back. The block-table entries of all of a thread's rows are fetched first, in one batch
 // of independent loads, and serve both the key and the value copy: looked up row by row, each
 // copy would wait a full memory round trip for its page id.
 template <int HEAD_DIM>
 __device__ __forceinline__ void load_tile(unsigned char* k_dst, unsigned char* v_dst, const int* table,
                                           const FlashParams& p, int kv_head, int value_head, int tile_start, int lo,
-                                          int hi) {
+                                          int hi, int keep) {
   constexpr int kChunks = HEAD_DIM / 8;
+  if constexpr (kFlashThreads % kChunks != 0) {
+    // A row's chunks do not divide the block: every copy works out its own row.
+    constexpr int kCopies = kTileKeys * kChunks / kFlashThreads;
+    static_assert(kTileKeys * kChunks % kFlashThreads == 0, "whole copies per thread");
+    const int page_size = p.page_mask + 1;
+    const int64_t v_shift = value_head >= 0 ? static_cast<int64_t>(value_head - kv_head) * page_size * HEAD_DIM : 0;
+#pragma unroll 4
+    for (int i = 0; i < kCopies; ++i) {
+      const int idx = threadIdx.x + i * kFlashThreads;
+      const int row = idx / kChunks, chunk = idx - row * kChunks;
+      const int key = tile_start + row;
+      const bool wanted = (key >= lo && key <= hi) || key < keep;
+      const int page = wanted ? __ldg(table + (key >> p.page_shift)) : -1;
+      const bool valid = wanted && page >= 0 && page < p.num_pages;
+      if (wanted && !valid) atomicOr(p.err, ERRBIT_BAD_PAGE);
+      const int64_t offset = valid ? ((static_cast<int64_t>(page) * p.kv_heads + kv_head) * page_size + (key & p.page_mask)) * HEAD_DIM + chunk * 8 : 0;
+      cp_async_16(smem_u32(k_dst + tile_offset<HEAD_DIM>(row, chunk)), p.k_arena + offset, valid);
+      cp_async_16(smem_u32(v_dst + tile_offset<HEAD_DIM>(row, chunk)), p.v_arena + offset + (valid ? v_shift : 0), valid);
+    }
+    return;
+  }
   constexpr int kRowsPerPass = kFlashThreads / kChunks;
   constexpr int kPasses = kTileKeys / kRowsPerPass;
   const int chunk = threadIdx.x % kChunks;
@@ -146,7 +178,7 @@ __device__ __forceinline__ void load_tile(unsigned char* k_dst, unsigned char* v
   if (page_size >= kTileKeys) {
     // The whole tile lies in one page (tiles start at multiples of 64 and the page size is a
     // power of two): one table entry, then a fixed stride from row to row.
-    const bool any = tile_start + kTileKeys - 1 >= lo && tile_start <= hi;
+    const bool any = (tile_start + kTileKeys - 1 >= lo && tile_start <= hi) || tile_start < keep;
     const int page = any ? __ldg(table + (tile_start >> p.page_shift)) : 0;
     const bool page_ok = page >= 0 && page < p.num_pages;
     if (any && !page_ok) atomicOr(p.err, ERRBIT_BAD_PAGE);
@@ -157,7 +189,7 @@ __device__ __forceinline__ void load_tile(unsigned char* k_dst, unsigned char* v
     for (int pass = 0; pass < kPasses; ++pass) {
       const int row = row0 + pass * kRowsPerPass;
       const int key = tile_start + row;
-      const bool valid = page_ok && key >= lo && key <= hi;
+      const bool valid = page_ok && ((key >= lo && key <= hi) || key < keep);
       const int64_t offset = valid ? base + static_cast<int64_t>(pass) * kRowsPerPass * HEAD_DIM : 0;
       cp_async_16(smem_u32(k_dst + tile_offset<HEAD_DIM>(row, chunk)), p.k_arena + offset, valid);
       cp_async_16(smem_u32(v_dst + tile_offset<HEAD_DIM>(row, chunk)), p.v_arena + offset + (valid ? v_shift : 0), valid);
@@ -168,13 +200,13 @@ __device__ __forceinline__ void load_tile(unsigned char* k_dst, unsigned char* v
 #pragma unroll
   for (int pass = 0; pass < kPasses; ++pass) {
     const int key = tile_start + row0 + pass * kRowsPerPass;
-    pages[pass] = (key >= lo && key <= hi) ? __ldg(table + (key >> p.page_shift)) : -1;
+    pages[pass] = ((key >= lo && key <= hi) || key < keep) ? __ldg(table + (key >> p.page_shift)) : -1;
   }
 #pragma unroll
   for (int pass = 0; pass < kPasses; ++pass) {
     const int row = row0 + pass * kRowsPerPass;
     const int key = tile_start + row;
-    const bool in_range = key >= lo && key <= hi;
+    const bool in_range = (key >= lo && key <= hi) || key < keep;
     const int page = pages[pass];
     bool valid = in_range && page >= 0 && page < p.num_pages;
     if (in_range && !valid) atomicOr(p.err, ERRBIT_BAD_PAGE);
@@ -335,11 +367,15 @@ __device__ __forceinline__ void finish_decode_block(const FlashParams& p, unsign
   cluster_sync_all();  // nobody leaves while its shared memory is still being read
 }
 
-// SHAPED: scores pass `shaped_score` (soft cap, bias by distance) and a query sees only the keys of its own chunk of
-// positions; the other instantiations carry none of that code.
-template <int HEAD_DIM, bool DECODE, bool SHAPED = false>
+// FORM_SHAPED: scores pass `shaped_score` (soft cap, bias by distance) and a query sees only the keys of its own chunk of
+// positions. FORM_KEPT: the first `keep_first` keys stay visible in front of the window. FORM_SIGMOID: the same visible
+// keys, each weighing sigmoid(score + bias of the head). The other instantiations carry none of that code.
+template <int HEAD_DIM, bool DECODE, int FORM = FORM_SOFTMAX>
 __global__ void __launch_bounds__(kFlashThreads)
 paged_flash_attention_kernel(const FlashParams p) {
+  constexpr bool SHAPED = FORM == FORM_SHAPED;
+  constexpr bool SIGMOID = FORM == FORM_SIGMOID;
+  constexpr bool KEPT = FORM == FORM_KEPT || SIGMOID;
   constexpr int kKSteps = HEAD_DIM / 16;   // k-steps of the score product
   constexpr int kDimTiles = HEAD_DIM / 8;  // n-tiles of the output
   constexpr int kTileBytes = kTileKeys * HEAD_DIM * 2;
@@ -392,6 +428,11 @@ paged_flash_attention_kernel(const FlashParams p) {
   if (SHAPED && chunk > 0) lo = max(lo, (first_pos + block_first_token) / chunk * chunk);  // the block's first row sees furthest back
   int hi = first_pos + block_last_token;  // inclusive
   int tile_begin = lo / kTileKeys, tile_end = hi / kTileKeys + 1;
+  // The walk counts tiles: first the kept keys' tiles that the window's do not cover, then the window's.
+  const int keep = KEPT && p.window > 0 ? min(p.keep_first, lo) : 0;
+  const int kept_tiles = min((keep + kTileKeys - 1) / kTileKeys, tile_begin);
+  const int window_tile = tile_begin;
+  tile_begin -= kept_tiles;
   if (DECODE && p.splits > 1) {
     const int tiles = tile_end - tile_begin;
     const int per_split = max(min_tiles_per_split(p.splits), (tiles + p.splits - 1) / p.splits);
@@ -399,6 +440,10 @@ paged_flash_attention_kernel(const FlashParams p) {
     tile_end = min(tile_end, tile_begin + per_split);
   }
   const int num_tiles = max(0, tile_end - tile_begin);
+  auto start_of = [&](int it) {  // first key of the block's tile `it`
+    const int t = tile_begin + it;
+    return (KEPT && t < window_tile ? t - (window_tile - kept_tiles) : t) * kTileKeys;
+  };
 
   // This thread's two rows (r0 = lane / 4 and r0 + 8 of the warp's block).
   const int r0 = row_base + (lane >> 2), r1 = r0 + 8;
@@ -416,6 +461,8 @@ paged_flash_attention_kernel(const FlashParams p) {
 #pragma unroll
   for (int i = 0; i < kDimTiles; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
+  const float gate0 = SIGMOID && live0 ? __ldg(p.shape.sigmoid_bias + head0) * kLog2e : 0.f;
+  const float gate1 = SIGMOID && live1 ? __ldg(p.shape.sigmoid_bias + head1) * kLog2e : 0.f;
 
   // Fill the ring. Tiles that hold only keys of earlier steps are requested before the wait
   // for the kernel in front (decode only); they always come first in the block's range. Every
@@ -423,11 +470,11 @@ paged_flash_attention_kernel(const FlashParams p) {
   auto fetch = [&](int it) {
     const int slot = it % kRing;
     load_tile<HEAD_DIM>(k_tiles + slot * kTileBytes, v_tiles + slot * kTileBytes, table, p, kv_head, value_head,
-                        (tile_begin + it) * kTileKeys, lo, hi);
+                        start_of(it), lo, hi, keep);
   };
   int issued = 0;
   if (DECODE) {
-    while (issued < kRing && issued < num_tiles && (tile_begin + issued + 1) * kTileKeys <= first_pos) {
+    while (issued < kRing && issued < num_tiles && start_of(issued) + kTileKeys <= first_pos) {
       fetch(issued);
       cp_async_commit();
       ++issued;
@@ -457,7 +504,7 @@ paged_flash_attention_kernel(const FlashParams p) {
 
   for (int it = 0; it < num_tiles; ++it) {
     const int stage = it % kRing;
-    const int tile_start = (tile_begin + it) * kTileKeys;
+    const int tile_start = start_of(it);
     // One group is committed per iteration, so all but the newest kRing - 1 have landed.
     cp_async_wait<kRing - 1>();
     __syncthreads();
@@ -505,9 +552,10 @@ paged_flash_attention_kernel(const FlashParams p) {
           const int key = key_base + n * 8 + (lane & 3) * 2 + (e & 1);
           const int pos = e < 2 ? pos0 : pos1;
           if (SHAPED) v = shaped_score_fast(s[n][e], p, e < 2 ? bias0 : bias1, pos - key, far_tile, e < 2 ? far_bias0 : far_bias1);
+          if (SIGMOID) v += e < 2 ? gate0 : gate1;
           if (tile_needs_mask) {
             const bool live = e < 2 ? live0 : live1;
-            const bool visible = live && key <= pos && key >= lo && (p.window == 0 || key > pos - p.window) &&
+            const bool visible = live && key <= pos && ((key >= lo && (p.window == 0 || key > pos - p.window)) || (KEPT && key < p.keep_first)) &&
                                  (!SHAPED || key >= (e < 2 ? chunk_lo0 : chunk_lo1));
             if (!visible) v = -INFINITY;
           }
@@ -516,6 +564,14 @@ paged_flash_attention_kernel(const FlashParams p) {
           else tile_max1 = fmaxf(tile_max1, v);
         }
       }
+      uint32_t pf[kGroups][4];
+      if constexpr (SIGMOID) {
+#pragma unroll
+        for (int n = 0; n < 2 * kGroups; ++n) {
+          pf[n >> 1][(n & 1) * 2 + 0] = pack_bf16(sigmoid_base2(s[n][0]), sigmoid_base2(s[n][1]));
+          pf[n >> 1][(n & 1) * 2 + 1] = pack_bf16(sigmoid_base2(s[n][2]), sigmoid_base2(s[n][3]));
+        }
+      } else {
       tile_max0 = fmaxf(tile_max0, __shfl_xor_sync(0xffffffffu, tile_max0, 1));
       tile_max0 = fmaxf(tile_max0, __shfl_xor_sync(0xffffffffu, tile_max0, 2));
       tile_max1 = fmaxf(tile_max1, __shfl_xor_sync(0xffffffffu, tile_max1, 1));
@@ -526,7 +582,6 @@ paged_flash_attention_kernel(const FlashParams p) {
       m0 = new0;
       m1 = new1;
       float sum0 = 0.f, sum1 = 0.f;
-      uint32_t pf[kGroups][4];
 #pragma unroll
       for (int n = 0; n < 2 * kGroups; ++n) {
         const float p00 = exp2f(s[n][0] - use0), p01 = exp2f(s[n][1] - use0);
@@ -547,6 +602,7 @@ paged_flash_attention_kernel(const FlashParams p) {
           o[i][2] *= alpha1;
           o[i][3] *= alpha1;
         }
+      }
       }
       // O += P V over the warp's keys, 16 at a time.
       {
@@ -576,6 +632,11 @@ paged_flash_attention_kernel(const FlashParams p) {
   l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
   l1 += __shfl_xor_sync(0xffffffffu, l1, 1);
   l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
+  if (SIGMOID) {
+    // Nothing is normalised. The merges divide by the sum of l * 2^m over the four warps and the splits: that sum is 1.
+    m0 = m1 = 0.f;
+    l0 = l1 = DECODE ? 1.f / static_cast<float>(kWarps * p.splits) : 1.f;
+  }
 
   const int col = (lane & 3) * 2;
   if (!DECODE) {
@@ -970,16 +1031,16 @@ constexpr size_t flash_smem_bytes(bool decode) {
   return tiles > merge ? tiles : merge;
 }
 
-template <int HEAD_DIM, bool SHAPED>
+template <int HEAD_DIM, int FORM>
 int launch_flash(const FlashParams& p, int num_seqs, int decode, int max_q_len, int tokens,
                  cudaStream_t stream) {
   const size_t smem = flash_smem_bytes<HEAD_DIM>(decode != 0);
   static bool configured = false;
   if (!configured) {
-    cudaError_t a = cudaFuncSetAttribute(paged_flash_attention_kernel<HEAD_DIM, true, SHAPED>,
+    cudaError_t a = cudaFuncSetAttribute(paged_flash_attention_kernel<HEAD_DIM, true, FORM>,
                                          cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          static_cast<int>(flash_smem_bytes<HEAD_DIM>(true)));
-    cudaError_t b = cudaFuncSetAttribute(paged_flash_attention_kernel<HEAD_DIM, false, SHAPED>,
+    cudaError_t b = cudaFuncSetAttribute(paged_flash_attention_kernel<HEAD_DIM, false, FORM>,
                                          cudaFuncAttributeMaxDynamicSharedMemorySize,
                                          static_cast<int>(flash_smem_bytes<HEAD_DIM>(false)));
     if (a != cudaSuccess || b != cudaSuccess) return b200_fail("flash attention: cannot size shared memory");
@@ -991,7 +1052,7 @@ int launch_flash(const FlashParams& p, int num_seqs, int decode, int max_q_len, 
     if (p.splits > 1 && p.cluster_merge) {
       static bool wide_clusters = false;
       if (p.splits > 8 && !wide_clusters) {
-        if (cudaFuncSetAttribute(paged_flash_attention_kernel<HEAD_DIM, true, SHAPED>,
+        if (cudaFuncSetAttribute(paged_flash_attention_kernel<HEAD_DIM, true, FORM>,
                                  cudaFuncAttributeNonPortableClusterSizeAllowed, 1) != cudaSuccess)
           return b200_fail("flash attention: clusters of %d blocks are not allowed here", p.splits);
         wide_clusters = true;
@@ -1010,18 +1071,18 @@ int launch_flash(const FlashParams& p, int num_seqs, int decode, int max_q_len, 
       attributes[1].val.programmaticStreamSerializationAllowed = 1;
       config.attrs = attributes;
       config.numAttrs = b200_overlap_enabled() ? 2 : 1;
-      const cudaError_t status = cudaLaunchKernelEx(&config, paged_flash_attention_kernel<HEAD_DIM, true, SHAPED>, p);
+      const cudaError_t status = cudaLaunchKernelEx(&config, paged_flash_attention_kernel<HEAD_DIM, true, FORM>, p);
       if (status != cudaSuccess) return b200_fail("flash attention: %s", cudaGetErrorString(status));
       return 0;
     }
-    launch_kernel(paged_flash_attention_kernel<HEAD_DIM, true, SHAPED>, grid, dim3(kFlashThreads), smem, stream, p);
+    launch_kernel(paged_flash_attention_kernel<HEAD_DIM, true, FORM>, grid, dim3(kFlashThreads), smem, stream, p);
     if (p.splits > 1) {
       launch_merge<HEAD_DIM>(p.partial_out, p.partial_ml, p.out, planes * tokens * p.q_heads, p.splits, stream);
     }
   } else {
     const int row_blocks = (max_q_len * p.group + kWarps * 16 - 1) / (kWarps * 16);
     const dim3 grid(row_blocks, p.kv_heads, num_seqs);
-    launch_kernel(paged_flash_attention_kernel<HEAD_DIM, false, SHAPED>, grid, dim3(kFlashThreads), smem, stream, p);
+    launch_kernel(paged_flash_attention_kernel<HEAD_DIM, false, FORM>, grid, dim3(kFlashThreads), smem, stream, p);
   }
   return b200_check_launch("paged_flash_attention");
 }
@@ -1064,7 +1125,7 @@ size_t decode_tma_smem_bytes(int stages) {
 // Whether the tuned kernel takes this shape; the caller uses the plain kernel otherwise.
 B200_API int b200_flash_attention_supported(int q_heads, int kv_heads, int head_dim, int page_size,
                                             int decode) {
-  if (head_dim != 64 && head_dim != 128) return 0;
+  if (head_dim != 64 && head_dim != 128 && head_dim != 192) return 0;
   if (q_heads % kv_heads) return 0;
   if (page_size <= 0 || (page_size & (page_size - 1))) return 0;
   if (decode && q_heads / kv_heads > 16) return 0;
@@ -1087,12 +1148,14 @@ B200_API int b200_paged_flash_attention(const void* q, const void* k_arena, cons
                                         const int* seq_q_len, const int* seq_kv_len, int first_seq,
                                         int num_seqs, int tokens, int max_q_len, int max_pages,
                                         int num_pages, int q_heads, int kv_heads, int head_dim,
-                                        int page_size, int window, float scale, int decode, int splits,
+                                        int page_size, int window, int keep_first, float scale, int decode, int splits,
                                         int value_head, float softcap, const float* bias, int bias_reach, int chunk,
-                                        float* scratch, int* err, cudaStream_t stream) {
+                                        const float* sigmoid_bias, float* scratch, int* err, cudaStream_t stream) {
   if (num_seqs == 0) return 0;
   B200_REQUIRE(softcap >= 0.f && chunk >= 0 && (bias == nullptr || bias_reach >= 0), "paged_flash_attention: bad score shape");
   const bool shaped = softcap > 0.f || bias != nullptr || chunk > 0;
+  B200_REQUIRE(keep_first >= 0 && !(shaped && (sigmoid_bias != nullptr || (window > 0 && keep_first > 0))),
+               "paged_flash_attention: capped, biased or chunked scores go with a plain softmax over one range of keys");
   const bool every_value_head = value_head == kEveryValueHead;
   B200_REQUIRE(value_head < kv_heads, "paged_flash_attention: value head %d of %d", value_head, kv_heads);
   B200_REQUIRE(!every_value_head || (decode && first_seq == 0 && kv_heads * kv_heads <= 65535),
@@ -1124,24 +1187,29 @@ B200_API int b200_paged_flash_attention(const void* q, const void* k_arena, cons
   p.page_shift = shift;
   p.page_mask = page_size - 1;
   p.window = window;
+  p.keep_first = keep_first;
   p.splits = decode ? splits : 1;
   p.cluster_merge = (scratch == nullptr && p.splits > 1) ? 1 : 0;
   p.value_head = every_value_head ? -1 : value_head;
   p.plane_tokens = every_value_head ? tokens : 0;
   p.scale_log2 = scale * kLog2e;
   p.scale = scale;
-  p.shape = ScoreShape{softcap, bias, bias_reach, chunk};
+  p.shape = ScoreShape{softcap, bias, bias_reach, chunk, sigmoid_bias};
   p.cap_twice_inv = softcap > 0.f ? 2.f / softcap : 0.f;
   p.err = err;
   p.partial_out = scratch;
   const int64_t planes = every_value_head ? kv_heads : 1;
   p.partial_ml = scratch ? scratch + planes * tokens * q_heads * p.splits * head_dim : nullptr;
-  if (shaped) {
-    if (head_dim == 64) return launch_flash<64, true>(p, num_seqs, decode, max_q_len, tokens, stream);
-    return launch_flash<128, true>(p, num_seqs, decode, max_q_len, tokens, stream);
-  }
-  if (head_dim == 64) return launch_flash<64, false>(p, num_seqs, decode, max_q_len, tokens, stream);
-  return launch_flash<128, false>(p, num_seqs, decode, max_q_len, tokens, stream);
+  auto launch = [&](auto dim) {
+    constexpr int kDim = decltype(dim)::value;
+    if (shaped) return launch_flash<kDim, FORM_SHAPED>(p, num_seqs, decode, max_q_len, tokens, stream);
+    if (sigmoid_bias != nullptr) return launch_flash<kDim, FORM_SIGMOID>(p, num_seqs, decode, max_q_len, tokens, stream);
+    if (window > 0 && keep_first > 0) return launch_flash<kDim, FORM_KEPT>(p, num_seqs, decode, max_q_len, tokens, stream);
+    return launch_flash<kDim, FORM_SOFTMAX>(p, num_seqs, decode, max_q_len, tokens, stream);
+  };
+  if (head_dim == 64) return launch(std::integral_constant<int, 64>{});
+  if (head_dim == 128) return launch(std::integral_constant<int, 128>{});
+  return launch(std::integral_constant<int, 192>{});
 }
 
 // Shapes the TMA-fed decode kernel takes: head_dim 128, pages of at least 64 rows (a 64-key
@@ -1196,13 +1264,14 @@ B200_API int b200_paged_decode_attention_tma(const void* q, const void* k_arena,
   p.page_shift = shift;
   p.page_mask = page_size - 1;
   p.window = window;
+  p.keep_first = 0;
   p.splits = splits;
   p.cluster_merge = (scratch == nullptr && splits > 1) ? 1 : 0;
   p.value_head = -1;
   p.plane_tokens = 0;
   p.scale_log2 = scale * kLog2e;
   p.scale = scale;
-  p.shape = ScoreShape{0.f, nullptr, 0, 0};
+  p.shape = ScoreShape{0.f, nullptr, 0, 0, nullptr};
   p.cap_twice_inv = 0.f;
   p.err = err;
   p.partial_out = scratch;

@@ -11,7 +11,9 @@
 //
 // Beyond the scale a score may be shaped (ScoreShape in common.cuh): soft-capped, s <- cap * tanh(s / cap); given a
 // learned bias by the key's distance, read from a table [q_heads][reach + 1] at min(pos - key, reach) and added after
-// the cap; and restricted to the query's own chunk of positions, keys from floor(pos / chunk) * chunk on.
+// the cap; and restricted to the query's own chunk of positions, keys from floor(pos / chunk) * chunk on. With
+// `sigmoid_bias` a visible key weighs sigmoid(score + bias of the head) and nothing is normalised. With a window the
+// first `keep_first` keys of the request stay visible in front of it.
 #include "common.cuh"
 
 namespace {
@@ -55,8 +57,8 @@ paged_attention_plain_kernel(const T* __restrict__ q, const T* __restrict__ k_ar
                              const int* __restrict__ token_seq,
                              const int* __restrict__ block_table, int max_pages, int num_pages,
                              T* __restrict__ out, int q_heads, int kv_heads, int head_dim,
-                             int page_size, int window, float scale, int value_head, const ScoreShape shape,
-                             int* __restrict__ err) {
+                             int page_size, int window, int keep_first, float scale, int value_head,
+                             const ScoreShape shape, int* __restrict__ err) {
   extern __shared__ __align__(16) unsigned char smem_raw[];
   float* qs = reinterpret_cast<float*>(smem_raw);                  // [head_dim]
   float* probs = qs + head_dim;                                    // [kThreads]
@@ -83,8 +85,14 @@ paged_attention_plain_kernel(const T* __restrict__ q, const T* __restrict__ k_ar
   for (int i = 0; i < kMaxDimsPerThread; ++i) acc[i] = 0.f;
   float running_max = -INFINITY, running_sum = 0.f;
 
-  for (int k0 = lo; k0 <= pos; k0 += kThreads) {
-    const int j = k0 + tid;
+  // The walk counts visible keys: the kept ones in front of the window, then lo .. pos.
+  const int kept = window > 0 ? min(keep_first, lo) : 0;
+  const int visible = kept + pos - lo + 1;
+  const bool sigmoid = shape.sigmoid_bias != nullptr;
+  const float sigmoid_bias = sigmoid ? shape.sigmoid_bias[h] : 0.f;
+  for (int k0 = 0; k0 < visible; k0 += kThreads) {
+    const int walk = k0 + tid;
+    const int j = walk < kept ? walk : (walk < visible ? walk - kept + lo : pos + 1);
     float s = -INFINITY;
     int64_t off = -1;
     if (j <= pos) {
@@ -100,14 +108,15 @@ paged_attention_plain_kernel(const T* __restrict__ q, const T* __restrict__ k_ar
     offsets[tid] = off;
     const float chunk_max = block_max(s, scratch);
     const float new_max = fmaxf(running_max, chunk_max);
-    const float p = (off >= 0 && new_max > -INFINITY) ? expf(s - new_max) : 0.f;
+    float p = (off >= 0 && new_max > -INFINITY) ? expf(s - new_max) : 0.f;
+    if (sigmoid) p = off >= 0 ? 1.f / (1.f + expf(-(s + sigmoid_bias))) : 0.f;
     probs[tid] = p;
     const float chunk_sum = block_sum(p, scratch);
-    const float alpha = (running_max > -INFINITY) ? expf(running_max - new_max) : 0.f;
+    const float alpha = sigmoid ? 1.f : ((running_max > -INFINITY) ? expf(running_max - new_max) : 0.f);
     running_sum = running_sum * alpha + chunk_sum;
     running_max = new_max;
     __syncthreads();
-    const int count = min(kThreads, pos - k0 + 1);
+    const int count = min(kThreads, visible - k0);
 #pragma unroll
     for (int i = 0; i < kMaxDimsPerThread; ++i) {
       const int d = tid + i * kThreads;
@@ -123,7 +132,7 @@ paged_attention_plain_kernel(const T* __restrict__ q, const T* __restrict__ k_ar
     __syncthreads();
   }
   T* orow = out + (static_cast<int64_t>(t) * q_heads + h) * head_dim;
-  const float inv = running_sum > 0.f ? 1.f / running_sum : 0.f;
+  const float inv = sigmoid ? 1.f : (running_sum > 0.f ? 1.f / running_sum : 0.f);
 #pragma unroll
   for (int i = 0; i < kMaxDimsPerThread; ++i) {
     const int d = tid + i * kThreads;
@@ -137,19 +146,19 @@ B200_API int b200_paged_attention_plain(const void* q, const void* k_arena, cons
                                         const int* positions, const int* token_seq,
                                         const int* block_table, int max_pages, int num_pages,
                                         void* out, int tokens, int q_heads, int kv_heads,
-                                        int head_dim, int page_size, int window, float scale,
+                                        int head_dim, int page_size, int window, int keep_first, float scale,
                                         int value_head, float softcap, const float* bias, int bias_reach, int chunk,
-                                        int dtype, int* err, cudaStream_t stream) {
+                                        const float* sigmoid_bias, int dtype, int* err, cudaStream_t stream) {
   if (tokens == 0) return 0;
   B200_REQUIRE(softcap >= 0.f && chunk >= 0 && (bias == nullptr || bias_reach >= 0), "paged_attention_plain: bad score shape");
-  const ScoreShape shape{softcap, bias, bias_reach, chunk};
+  const ScoreShape shape{softcap, bias, bias_reach, chunk, sigmoid_bias};
   B200_REQUIRE(tokens > 0 && q_heads > 0 && kv_heads > 0 && q_heads % kv_heads == 0,
                "paged_attention_plain: %d query heads over %d kv heads", q_heads, kv_heads);
   B200_REQUIRE(head_dim > 0 && head_dim % 8 == 0 && head_dim <= kThreads * kMaxDimsPerThread,
                "paged_attention_plain: head_dim %d must be a multiple of 8, at most %d", head_dim,
                kThreads * kMaxDimsPerThread);
   B200_REQUIRE(q_heads <= 65535, "paged_attention_plain: too many heads");
-  B200_REQUIRE(page_size > 0 && max_pages > 0 && window >= 0, "paged_attention_plain: bad geometry");
+  B200_REQUIRE(page_size > 0 && max_pages > 0 && window >= 0 && keep_first >= 0, "paged_attention_plain: bad geometry");
   B200_REQUIRE(value_head < kv_heads, "paged_attention_plain: value head %d of %d", value_head, kv_heads);
   const dim3 grid(tokens, q_heads);
   const size_t smem = sizeof(float) * (head_dim + kThreads) + sizeof(int64_t) * kThreads;
@@ -157,14 +166,14 @@ B200_API int b200_paged_attention_plain(const void* q, const void* k_arena, cons
     paged_attention_plain_kernel<float><<<grid, kThreads, smem, stream>>>(
         static_cast<const float*>(q), static_cast<const float*>(k_arena),
         static_cast<const float*>(v_arena), positions, token_seq, block_table, max_pages,
-        num_pages, static_cast<float*>(out), q_heads, kv_heads, head_dim, page_size, window, scale,
+        num_pages, static_cast<float*>(out), q_heads, kv_heads, head_dim, page_size, window, keep_first, scale,
         value_head, shape, err);
   } else if (dtype == DTYPE_BF16) {
     paged_attention_plain_kernel<__nv_bfloat16><<<grid, kThreads, smem, stream>>>(
         static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(k_arena),
         static_cast<const __nv_bfloat16*>(v_arena), positions, token_seq, block_table, max_pages,
         num_pages, static_cast<__nv_bfloat16*>(out), q_heads, kv_heads, head_dim, page_size,
-        window, scale, value_head, shape, err);
+        window, keep_first, scale, value_head, shape, err);
   } else {
     return b200_fail("paged_attention_plain: unknown dtype %d", dtype);
   }

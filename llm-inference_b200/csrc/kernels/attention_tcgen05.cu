@@ -14,7 +14,9 @@
 // before its product is issued), and no thread computes addresses row by row. Three S buffers
 // let the tensor core run two tiles ahead of each softmax group. Masking follows
 // python/instinct/batches.py:110-113: key <= query position and, with a window,
-// key > position - window.
+// key > position - window. Behind a window the first `keep_first` keys of a request may stay
+// visible (KEPT): the walk takes their tiles first, then the window's. SIGMOID turns a score into
+// a weight by a sigmoid: no maximum, no sum, nothing the two softmax groups have to agree on.
 //
 // Every wait (mbarriers, and the shared-memory word the two softmax threads of a row pass the
 // turn with) is bounded; on a timeout the block records ERRBIT_TIMEOUT, skips its further waits,
@@ -55,6 +57,8 @@ struct PrefillParams {
   int page_size, page_shift;
   int piece_rows;  // rows per TMA box: min(page_size, 128)
   int window;
+  int keep_first;  // the KEPT and SIGMOID forms only: the first this many keys stay visible in front of the window
+  const float* sigmoid_bias;  // [q_heads], the SIGMOID form only
   int value_head;  // >= 0: every block takes its values from this kv head's rows of the pages (keys stay its own)
   float scale_log2;
   // The capped form only: scores pass cap * tanh(score / cap) and a query sees only the keys of its own chunk.
@@ -210,8 +214,9 @@ __device__ __forceinline__ float capped_exponent(float raw, const PrefillParams&
 // of the head (plus the one number that serves a tile wholly beyond the bias's reach): probabilities stay below
 // 2^kSlack as before and fall short of it by the spread of the head's biases at most. The biases themselves are read
 // in the second pass only, and only in tiles within reach.
-// Three instantiations: plain, CAPPED (cap and chunks) and CAPPED with BIASED.
-template <bool CAPPED, bool BIASED>
+// KEPT and SIGMOID: see the top. Five instantiations: plain, CAPPED (cap and chunks), CAPPED with BIASED, KEPT, SIGMOID (which
+// is KEPT too).
+template <bool CAPPED, bool BIASED, bool KEPT = false, bool SIGMOID = false>
 __global__ void __launch_bounds__(kThreadsA, 1)
 flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map,
                              const PrefillParams p) {
@@ -258,8 +263,12 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap k_map, const __
   int lo = p.window > 0 ? max(0, first_pos + first_token - p.window + 1) : 0;
   if (CAPPED && p.chunk > 0) lo = max(lo, (first_pos + first_token) / p.chunk * p.chunk);  // the first row sees furthest back
   const int hi = first_pos + last_token;  // inclusive
-  const int tile_begin = lo / kKeys, tile_end = hi / kKeys + 1;
-  const int num_tiles = tile_end - tile_begin;
+  const int tile_end = hi / kKeys + 1;
+  // The walk counts tiles: first the kept keys' tiles that the window's do not cover, then the window's.
+  const int window_tile = lo / kKeys;
+  const int kept_tiles = KEPT && p.window > 0 ? min((min(p.keep_first, lo) + kKeys - 1) / kKeys, window_tile) : 0;
+  const int num_tiles = kept_tiles + tile_end - window_tile;
+  auto start_of = [&](int it) { return (KEPT && it < kept_tiles ? it : window_tile + it - kept_tiles) * kKeys; };
   const int pieces_per_tile = kKeys / p.piece_rows;
   if (num_tiles * pieces_per_tile > kMaxChunks) {
     // The launcher sized the walk from the host's lengths; lengths on the device that exceed
@@ -296,7 +305,7 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap k_map, const __
   // this may precede the wait for the kernel in front (which wrote the queries and the newest
   // keys).
   for (int i = threadIdx.x; i < num_tiles * pieces_per_tile; i += kThreadsA) {
-    const int key = tile_begin * kKeys + i * p.piece_rows;
+    const int key = start_of(i / pieces_per_tile) + i % pieces_per_tile * p.piece_rows;
     // Pieces past the request's last key are read too (the table pads them with a page that
     // exists): their scores are masked, and their values only ever meet a probability of zero.
     pages[i] = (key >> p.page_shift) < p.max_pages ? table[key >> p.page_shift] : -1;
@@ -375,7 +384,7 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap k_map, const __
           if (leader) atomicOr(p.err, ERRBIT_BAD_PAGE);
           continue;
         }
-        const int key = (tile_begin + it) * kKeys + piece * p.piece_rows;
+        const int key = start_of(it) + piece * p.piece_rows;
         const int arena_row = (page * p.kv_heads + row_head) * p.page_size + (key & (p.page_size - 1));
         const int offset = piece * p.piece_rows * 128;
         if (leader) {
@@ -473,6 +482,7 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap k_map, const __
     const int q_head = kv_head * p.group + (row - (row / p.group) * p.group);
     const float* bias_row = BIASED ? p.bias + static_cast<int64_t>(q_head) * (p.bias_reach + 1) : nullptr;
     const float bias_peak = bias_row ? __ldg(p.bias_peak + q_head) * kLog2eA : 0.f;
+    const float gate_bias = SIGMOID && live ? __ldg(p.sigmoid_bias + q_head) * kLog2eA : 0.f;
     const float far_bias = bias_row ? __ldg(bias_row + p.bias_reach) * kLog2eA : 0.f;
     volatile int* next_tile = &row_next[r];
     volatile float* shared_m = &row_m[r];
@@ -490,13 +500,44 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap k_map, const __
     for (int it = group; it < num_tiles; it += 2) {
       if (ok && !__all_sync(0xffffffffu, bar_wait(&s_full[it % kScoreBuffers], (it / kScoreBuffers) & 1))) ok = false;
       fence_after();
-      const int tile_start = (tile_begin + it) * kKeys;
+      const int tile_start = start_of(it);
       const uint32_t s_addr = (tmem + (it % kScoreBuffers) * 128) + lane_addr;
       // Keys [rel_lo, rel_hi] of this tile are the ones this row attends to.
       const int rel_hi = live ? pos - tile_start : -1;
       int rel_lo = p.window > 0 ? pos - p.window + 1 - tile_start : 0;
       if (CAPPED && p.chunk > 0) rel_lo = max(rel_lo, pos / p.chunk * p.chunk - tile_start);
       const bool needs_mask = __any_sync(0xffffffffu, rel_hi < kKeys - 1 || rel_lo > 0);
+      // Keys of this tile in front of column rel_keep are visible whatever the window says.
+      const int rel_keep = KEPT && p.window > 0 ? p.keep_first - tile_start : 0;
+      auto hidden = [&](int c) { return c > rel_hi || (c < rel_lo && (!KEPT || c >= rel_keep)); };
+      if constexpr (SIGMOID) {
+        // P = sigmoid(s * scale + bias) in one pass; the look at PV[it - 2] keeps this thread's view of the o_done ring current.
+        if (it >= 2 && ok && !__all_sync(0xffffffffu, bar_wait(&o_done[(it - 2) & 3], ((it - 2) >> 2) & 1))) ok = false;
+        fence_after();
+#pragma unroll 1
+        for (int c0 = 0; c0 < kKeys; c0 += 32) {
+          uint32_t raw[32];
+          tmem_ld32(s_addr + c0, raw);
+          float w[32];
+#pragma unroll
+          for (int i = 0; i < 32; ++i) w[i] = fast_exp2(-fmaf(__uint_as_float(raw[i]), p.scale_log2, gate_bias));
+#pragma unroll
+          for (int i = 0; i < 32; ++i) w[i] = __fdividef(1.f, 1.f + w[i]);
+          if (needs_mask) {
+#pragma unroll
+            for (int i = 0; i < 32; ++i)
+              if (hidden(c0 + i)) w[i] = 0.f;
+          }
+          uint32_t packed[16];
+#pragma unroll
+          for (int i = 0; i < 32; i += 2) packed[i >> 1] = pack2(w[i], w[i + 1]);
+          tmem_st16((tmem + (it % kScoreBuffers) * 128) + lane_addr + (c0 >> 1), packed);
+        }
+        tmem_st_wait();
+        fence_before();
+        bar_arrive(&p_ready[it % kScoreBuffers]);
+        continue;
+      }
       // Two passes over the scores, 32 columns at a time (rolled loops: fully unrolled, this code
       // outgrew the instruction cache and the warps starved on fetches). Pass 1: the maximum.
       float mx0 = -INFINITY, mx1 = -INFINITY, mx2 = -INFINITY, mx3 = -INFINITY;
@@ -507,7 +548,7 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap k_map, const __
         if (needs_mask) {
 #pragma unroll
           for (int i = 0; i < 32; ++i)
-            if (c0 + i > rel_hi || c0 + i < rel_lo) raw[i] = 0xff800000u;  // -inf
+            if (hidden(c0 + i)) raw[i] = 0xff800000u;  // -inf
         }
 #pragma unroll
         for (int i = 0; i < 32; i += 4) {
@@ -589,7 +630,7 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap k_map, const __
         if (needs_mask) {
 #pragma unroll
           for (int i = 0; i < 32; ++i)
-            if (c0 + i > rel_hi || c0 + i < rel_lo) raw[i] = 0xff800000u;
+            if (hidden(c0 + i)) raw[i] = 0xff800000u;
         }
         if (CAPPED) {
           // Stage by stage over all 32 columns, so that each special-function operation has 31 independent ones beside it.
@@ -639,14 +680,18 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap k_map, const __
       bar_arrive(&p_ready[it % kScoreBuffers]);
     }
     // The finished row: O / l as bfloat16, l being both groups' sums brought to the final offset.
-    if (!turn_of(num_tiles)) ok = false;
-    {
-      const float m = *shared_m;
-      if (m != seen) l *= seen == -INFINITY ? 0.f : exp2f(seen - m);
+    if constexpr (SIGMOID) {
+      l = 1.f;  // nothing is normalised
+    } else {
+      if (!turn_of(num_tiles)) ok = false;
+      {
+        const float m = *shared_m;
+        if (m != seen) l *= seen == -INFINITY ? 0.f : exp2f(seen - m);
+      }
+      row_l[group][r] = l;
+      asm volatile("bar.sync 1, %0;" ::"n"(kSoftmaxThreads) : "memory");
+      l = row_l[0][r] + row_l[1][r];
     }
-    row_l[group][r] = l;
-    asm volatile("bar.sync 1, %0;" ::"n"(kSoftmaxThreads) : "memory");
-    l = row_l[0][r] + row_l[1][r];
     if (ok && num_tiles > 0) ok = bar_wait(&o_done[(num_tiles - 1) & 3], ((num_tiles - 1) >> 2) & 1);
     if (!ok && lane == 0) atomicOr(p.err, ERRBIT_TIMEOUT_A);
     fence_after();
@@ -734,9 +779,9 @@ B200_API int b200_flash_prefill_tcgen05(const void* q, const void* k_arena, cons
                                         const int* block_table, const int* seq_q_start, const int* seq_q_len,
                                         const int* seq_kv_len, int first_seq, int num_seqs, int max_q_len,
                                         int max_kv_len, int max_pages, int num_pages, int q_heads, int kv_heads,
-                                        int head_dim, int page_size, int window, float scale, int value_head, float softcap,
-                                        const float* bias, const float* bias_peak, int bias_reach, int chunk, int* err,
-                                        cudaStream_t stream) {
+                                        int head_dim, int page_size, int window, int keep_first, float scale, int value_head,
+                                        float softcap, const float* bias, const float* bias_peak, int bias_reach, int chunk,
+                                        const float* sigmoid_bias, int* err, cudaStream_t stream) {
   if (num_seqs == 0) return 0;
   B200_REQUIRE(softcap >= 0.f && chunk >= 0, "flash_prefill_tcgen05: bad cap or chunk");
   B200_REQUIRE(bias == nullptr || (bias_peak != nullptr && bias_reach >= 0), "flash_prefill_tcgen05: a bias by distance comes with its rows' maxima");
@@ -765,6 +810,8 @@ B200_API int b200_flash_prefill_tcgen05(const void* q, const void* k_arena, cons
   p.page_shift = shift;
   p.piece_rows = page_size < kKeys ? page_size : kKeys;
   p.window = window;
+  p.keep_first = keep_first;
+  p.sigmoid_bias = sigmoid_bias;
   p.value_head = value_head;
   p.scale_log2 = scale * kLog2eA;
   p.scale = scale;
@@ -775,6 +822,9 @@ B200_API int b200_flash_prefill_tcgen05(const void* q, const void* k_arena, cons
   p.bias_peak = bias_peak;
   p.bias_reach = bias_reach;
   const bool capped = softcap > 0.f || chunk > 0 || bias != nullptr;
+  const bool kept = window > 0 && keep_first > 0;
+  B200_REQUIRE(keep_first >= 0 && !(capped && (kept || sigmoid_bias != nullptr)),
+               "flash_prefill_tcgen05: capped, biased or chunked scores go with a plain softmax over one range of keys");
   CUtensorMap k_map, v_map;
   const int64_t rows = static_cast<int64_t>(num_pages) * kv_heads * page_size;
   if (arena_map(&k_map, k_arena, rows, p.piece_rows) != 0) return -1;
@@ -787,6 +837,10 @@ B200_API int b200_flash_prefill_tcgen05(const void* q, const void* k_arena, cons
         cudaFuncSetAttribute(flash_prefill_tcgen05_kernel<true, false>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                              static_cast<int>(smem)) != cudaSuccess ||
         cudaFuncSetAttribute(flash_prefill_tcgen05_kernel<true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                             static_cast<int>(smem)) != cudaSuccess ||
+        cudaFuncSetAttribute(flash_prefill_tcgen05_kernel<false, false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                             static_cast<int>(smem)) != cudaSuccess ||
+        cudaFuncSetAttribute(flash_prefill_tcgen05_kernel<false, false, true, true>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                              static_cast<int>(smem)) != cudaSuccess)
       return b200_fail("flash_prefill_tcgen05: cannot size shared memory (%zu bytes)", smem);
     configured = true;
@@ -796,6 +850,8 @@ B200_API int b200_flash_prefill_tcgen05(const void* q, const void* k_arena, cons
   const cudaError_t status =
       bias != nullptr ? launch_kernel(flash_prefill_tcgen05_kernel<true, true>, grid, dim3(kThreadsA), smem, stream, k_map, v_map, p)
       : capped        ? launch_kernel(flash_prefill_tcgen05_kernel<true, false>, grid, dim3(kThreadsA), smem, stream, k_map, v_map, p)
+      : sigmoid_bias  ? launch_kernel(flash_prefill_tcgen05_kernel<false, false, true, true>, grid, dim3(kThreadsA), smem, stream, k_map, v_map, p)
+      : kept          ? launch_kernel(flash_prefill_tcgen05_kernel<false, false, true>, grid, dim3(kThreadsA), smem, stream, k_map, v_map, p)
                       : launch_kernel(flash_prefill_tcgen05_kernel<false, false>, grid, dim3(kThreadsA), smem, stream, k_map, v_map, p);
   if (status != cudaSuccess) return b200_fail("flash_prefill_tcgen05: %s", cudaGetErrorString(status));
   return 0;

@@ -209,12 +209,14 @@ __device__ __forceinline__ float block_max(float v, float* scratch) {
 }
 
 // What an attention kernel does to a score beyond the scale: a soft cap, a learned bias by the key's distance and a
-// restriction to the query's own chunk of positions. All zero / null: nothing.
+// restriction to the query's own chunk of positions; and how a score becomes a weight (softmax, or a sigmoid per key).
+// All zero / null: nothing, and a softmax.
 struct ScoreShape {
   float softcap;      // > 0: s <- softcap * tanh(s / softcap)
   const float* bias;  // [q_heads][bias_reach + 1] by distance min(pos - key, bias_reach), added after the cap; null: none
   int bias_reach;
   int chunk;          // > 0: a query at `pos` sees keys from floor(pos / chunk) * chunk on only
+  const float* sigmoid_bias;  // [q_heads]: a visible key weighs sigmoid(score + bias of the head), nothing is normalised; null: softmax
 };
 
 // `s` is the scaled score, `bias_row` the query head's row of the bias table (or null), `distance` = pos - key >= 0.

@@ -7,10 +7,14 @@
 // be chosen; the `top` largest s among them are chosen (ties: the lower index), and their weights are
 // s / (sum of the chosen s + 1e-20) * scale. A second kind of router (`softmax_chosen`) scores an expert by its logit
 // itself, z plus a learned bias per expert, chooses the `top` largest and weighs them by the softmax over the chosen
-// logits only, times scale. A bias may be given to either kind.
+// logits only, times scale. A bias may be given to either kind. A third kind (`softmax_all`) scores an expert by the softmax
+// over all of them; the bias is a correction of the choice alone: it is added to the scores that compete (and a group
+// counts by the largest of its corrected scores), while a chosen expert's weight is its score itself times scale.
 //
 // Expert: g = min(W_gate h, limit), u = clamp(W_up h, -limit, limit), y = g sigmoid(1.702 g) (u + 1),
-// output W_down y. A limit of zero means the unclamped form y = silu(W_gate h) * (W_up h).
+// output W_down y. A limit of zero means the unclamped form y = silu(W_gate h) * (W_up h). An ungated expert has one
+// matrix in front: y = max(W_up h, 0)^2. The last of the experts the router chooses from may be identity experts, which
+// have no matrices: their slots are given no place, and the weighted sum takes the token's own input for them.
 //
 // Grouping: every (token, choice) pair is a slot. `moe_sort` (one block) counts the slots of each
 // expert, gives each expert a run of whole tiles of `tile_rows` sorted places (kTileM, or four times
@@ -19,6 +23,8 @@
 // rows share one expert's weights. Each output number is one thread's sum over K in a fixed order, so
 // a slot's result does not depend on which other slots share its tile, and the final sum over a
 // token's choices runs in the router's order: nothing depends on the batch.
+#include <type_traits>
+
 #include "common.cuh"
 
 namespace {
@@ -37,6 +43,11 @@ __device__ __forceinline__ float clamped_glu(float g, float u, float limit) {
   return g * sigmoid_f(1.702f * g) * (u + 1.f);
 }
 
+__device__ __forceinline__ float squared_relu(float u) {
+  u = fmaxf(u, 0.f);
+  return u * u;
+}
+
 // The lane holding the largest value (ties: the lowest index) among the lanes' candidates.
 __device__ __forceinline__ void warp_argmax(float& value, int& index) {
 #pragma unroll
@@ -50,24 +61,41 @@ __device__ __forceinline__ void warp_argmax(float& value, int& index) {
   }
 }
 
-// z [tokens][experts] -> ids [tokens][top], weights [tokens][top]. Shared memory per warp:
-// experts scores + groups group scores.
-__global__ void moe_route_kernel(const float* z, const float* __restrict__ bias, int softmax_chosen, int tokens, int experts, int groups,
+enum : int { ROUTE_SIGMOID = 0, ROUTE_SOFTMAX_CHOSEN = 1, ROUTE_SOFTMAX_ALL = 2 };
+
+// z [tokens][experts], rows `ld` apart -> ids [tokens][top], weights [tokens][top]. Shared memory per warp:
+// experts scores + groups group scores (+ experts weights, ROUTE_SOFTMAX_ALL).
+__global__ void moe_route_kernel(const float* z, int ld, const float* __restrict__ bias, int rule, int tokens, int experts, int groups,
                                  int keep, int top, float scale, int* ids, float* weights) {
   extern __shared__ float route_smem[];
+  const bool softmax_chosen = rule == ROUTE_SOFTMAX_CHOSEN, softmax_all = rule == ROUTE_SOFTMAX_ALL;
   wait_for_predecessor();
   let_successor_start();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
   const int t = blockIdx.x * warps + warp;
   if (t >= tokens) return;
-  float* s = route_smem + warp * (experts + groups);
+  float* s = route_smem + warp * ((softmax_all ? 2 : 1) * experts + groups);
   float* gs = s + experts;
+  float* score = gs + groups;  // ROUTE_SOFTMAX_ALL: what a chosen expert weighs
   const int size = experts / groups;
   for (int e = lane; e < experts; e += 32) {
-    const float logit = z[static_cast<int64_t>(t) * experts + e] + (bias ? bias[e] : 0.f);
-    s[e] = softmax_chosen ? logit : sigmoid_f(logit);
+    const float logit = z[static_cast<int64_t>(t) * ld + e] + (bias && !softmax_all ? bias[e] : 0.f);
+    s[e] = softmax_chosen || softmax_all ? logit : sigmoid_f(logit);
   }
   __syncwarp();
+  if (softmax_all) {
+    float largest = -INFINITY, total = 0.f;
+    for (int e = lane; e < experts; e += 32) largest = fmaxf(largest, s[e]);
+    largest = warp_max(largest);
+    for (int e = lane; e < experts; e += 32) total += expf(s[e] - largest);
+    total = warp_sum(total);
+    for (int e = lane; e < experts; e += 32) {
+      const float p = expf(s[e] - largest) / total;
+      score[e] = p;
+      s[e] = p + (bias ? bias[e] : 0.f);
+    }
+    __syncwarp();
+  }
   for (int g = lane; g < groups; g += 32) {
     float first = -INFINITY, second = -INFINITY;
     for (int i = 0; i < size; ++i) {
@@ -79,7 +107,7 @@ __global__ void moe_route_kernel(const float* z, const float* __restrict__ bias,
         second = v;
       }
     }
-    gs[g] = size > 1 ? first + second : first;
+    gs[g] = size > 1 && !softmax_all ? first + second : first;
   }
   __syncwarp();
   // Keep the best groups: the others' experts leave the contest.
@@ -106,6 +134,7 @@ __global__ void moe_route_kernel(const float* z, const float* __restrict__ bias,
       if (s[e] > best) best = s[e], at = e;
     warp_argmax(best, at);
     if (at >= experts) at = 0, best = 0.f;  // cannot happen with a valid configuration and finite logits
+    if (softmax_all) best = score[at];
     sum += best;
     if (lane == j % 32 && j < 32) mine = best, mine_id = at;
     if (j >= 32 && lane == 0) {  // more than 32 choices: written unnormalised, fixed up below
@@ -136,7 +165,7 @@ __global__ void moe_route_kernel(const float* z, const float* __restrict__ bias,
       for (int j = 32; j < top; ++j) weights[static_cast<int64_t>(t) * top + j] *= share;
     return;
   }
-  const float factor = scale / (sum + 1e-20f);
+  const float factor = softmax_all ? scale : scale / (sum + 1e-20f);
   if (lane < top) {
     ids[static_cast<int64_t>(t) * top + lane] = mine_id;
     weights[static_cast<int64_t>(t) * top + lane] = mine * factor;
@@ -179,11 +208,12 @@ __global__ void moe_sort_kernel(const int* ids, int slots, int experts, int capa
 }
 
 // act[place][n] = glu(h[token(place)] . W_gate[e][n], h . W_up[e][n]) for the tile's expert e.
-// w_gate_up [experts][2 * ff][width]: rows 0 .. ff are the gate's, the rest the up projection's.
+// w_gate_up [experts][2 * ff][width]: rows 0 .. ff are the gate's, the rest the up projection's. Ungated (mats = 1):
+// act = max(h . W_up[e][n], 0)^2 with w_up [experts][ff][width].
 template <typename T>
 __global__ void __launch_bounds__(kGemmThreads)
 moe_gate_up_kernel(const T* h, const T* __restrict__ weight, const int* place_slot, const int* tile_expert, const int* num_tiles, int top,
-                   int width, int ff, float limit, T* act) {
+                   int width, int ff, int mats, float limit, T* act) {
   __shared__ float a_tile[kTileM][kTileK + 1];
   __shared__ float g_tile[kTileN][kTileK + 1];
   __shared__ float u_tile[kTileN][kTileK + 1];
@@ -200,8 +230,8 @@ moe_gate_up_kernel(const T* h, const T* __restrict__ weight, const int* place_sl
     row_token[tid] = slot < 0 ? -1 : slot / top;
   }
   __syncthreads();
-  const T* wg = weight + static_cast<int64_t>(expert) * 2 * ff * width;
-  const T* wu = wg + static_cast<int64_t>(ff) * width;
+  const T* wg = weight + static_cast<int64_t>(expert) * mats * ff * width;
+  const T* wu = wg + (mats - 1) * static_cast<int64_t>(ff) * width;
   float acc_g[4] = {0.f, 0.f, 0.f, 0.f}, acc_u[4] = {0.f, 0.f, 0.f, 0.f};
   for (int k0 = 0; k0 < width; k0 += kTileK) {
     for (int idx = tid; idx < kTileM * kTileK; idx += kGemmThreads) {
@@ -232,7 +262,7 @@ moe_gate_up_kernel(const T* h, const T* __restrict__ weight, const int* place_sl
   for (int i = 0; i < 4; ++i) {
     const int r = ty * 4 + i;
     if (row_token[r] >= 0)
-      act[(static_cast<int64_t>(tile) * kTileM + r) * ff + n] = from_f32<T>(clamped_glu(acc_g[i], acc_u[i], limit));
+      act[(static_cast<int64_t>(tile) * kTileM + r) * ff + n] = from_f32<T>(mats == 1 ? squared_relu(acc_u[i]) : clamped_glu(acc_g[i], acc_u[i], limit));
   }
 }
 
@@ -323,7 +353,7 @@ __device__ __forceinline__ void mma_bf16(float (&d)[4], const uint32_t (&a)[4], 
 // acc[mat][m16 tile][n8 tile][4] of this warp's 32 rows (`warp_m`) and columns (`warp_n`); `b_rows[mat]` is row n0
 // of matrix `mat` ([.][K], K contiguous), `n_valid` how many of the kMmaN rows exist.
 template <int MATS, int MT>
-__device__ __forceinline__ void tile_product(const __nv_bfloat16* const* a_rows, const __nv_bfloat16* const (&b_rows)[MATS], int n_valid, int K,
+__device__ __forceinline__ void tile_product(const __nv_bfloat16* const* a_rows, const __nv_bfloat16* const* b_rows, int n_valid, int K,
                                              __nv_bfloat16 (*a_smem)[32 * MT][kMmaPitch], __nv_bfloat16 (*b_smem)[MATS][kMmaN][kMmaPitch],
                                              float (&acc)[MATS][2][MmaShape<MT>::n_tiles][4]) {
   using Shape = MmaShape<MT>;
@@ -391,14 +421,14 @@ __device__ __forceinline__ void tile_product(const __nv_bfloat16* const* a_rows,
   asm volatile("cp.async.wait_group 0;" ::: "memory");
 }
 
-template <int MT>
+template <int MT, int MATS>
 __global__ void __launch_bounds__(MmaShape<MT>::threads)
 moe_gate_up_mma_kernel(const __nv_bfloat16* h, const __nv_bfloat16* __restrict__ weight, const int* place_slot, const int* tile_expert,
                        const int* num_tiles, int top, int width, int ff, float limit, __nv_bfloat16* act) {
   using Shape = MmaShape<MT>;
   extern __shared__ __align__(16) unsigned char mma_smem[];
   auto a_smem = reinterpret_cast<__nv_bfloat16(*)[Shape::rows][kMmaPitch]>(mma_smem);
-  auto b_smem = reinterpret_cast<__nv_bfloat16(*)[2][kMmaN][kMmaPitch]>(mma_smem + sizeof(__nv_bfloat16) * kMmaStages * Shape::rows * kMmaPitch);
+  auto b_smem = reinterpret_cast<__nv_bfloat16(*)[MATS][kMmaN][kMmaPitch]>(mma_smem + sizeof(__nv_bfloat16) * kMmaStages * Shape::rows * kMmaPitch);
   __shared__ const __nv_bfloat16* a_rows[Shape::rows];
   wait_for_predecessor();
   let_successor_start();
@@ -411,10 +441,12 @@ moe_gate_up_mma_kernel(const __nv_bfloat16* h, const __nv_bfloat16* __restrict__
     a_rows[threadIdx.x] = slot < 0 ? nullptr : h + static_cast<int64_t>(slot / top) * width;
   }
   __syncthreads();
-  const __nv_bfloat16* wg = weight + (static_cast<int64_t>(expert) * 2 * ff + n0) * width;
-  const __nv_bfloat16* const b_rows[2] = {wg, wg + static_cast<int64_t>(ff) * width};
-  float acc[2][2][Shape::n_tiles][4];
-  tile_product<2, MT>(a_rows, b_rows, min(kMmaN, ff - n0), width, a_smem, b_smem, acc);
+  const __nv_bfloat16* wg = weight + (static_cast<int64_t>(expert) * MATS * ff + n0) * width;
+  const __nv_bfloat16* b_rows[MATS];
+#pragma unroll
+  for (int mat = 0; mat < MATS; ++mat) b_rows[mat] = wg + mat * static_cast<int64_t>(ff) * width;
+  float acc[MATS][2][Shape::n_tiles][4];
+  tile_product<MATS, MT>(a_rows, b_rows, min(kMmaN, ff - n0), width, a_smem, b_smem, acc);
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int warp_m = warp / Shape::warps_n, warp_n = warp % Shape::warps_n;
 #pragma unroll
@@ -426,8 +458,9 @@ moe_gate_up_mma_kernel(const __nv_bfloat16* h, const __nv_bfloat16* __restrict__
         const int r = warp_m * 32 + m * 16 + (lane >> 2) + half * 8;
         const int col = n0 + warp_n * (8 * Shape::n_tiles) + n * 8 + (lane & 3) * 2;
         if (a_rows[r] == nullptr || col >= ff) continue;  // ff is even: the pair is whole
-        const float y0 = clamped_glu(acc[0][m][n][half * 2], acc[1][m][n][half * 2], limit);
-        const float y1 = clamped_glu(acc[0][m][n][half * 2 + 1], acc[1][m][n][half * 2 + 1], limit);
+        const float g0 = acc[0][m][n][half * 2], g1 = acc[0][m][n][half * 2 + 1];
+        const float y0 = MATS == 1 ? squared_relu(g0) : clamped_glu(g0, acc[MATS - 1][m][n][half * 2], limit);
+        const float y1 = MATS == 1 ? squared_relu(g1) : clamped_glu(g1, acc[MATS - 1][m][n][half * 2 + 1], limit);
         *reinterpret_cast<__nv_bfloat162*>(act + (static_cast<int64_t>(tile) * Shape::rows + r) * ff + col) = __floats2bfloat162_rn(y0, y1);
       }
 }
@@ -472,18 +505,49 @@ moe_down_mma_kernel(const __nv_bfloat16* act, const __nv_bfloat16* __restrict__ 
       }
 }
 
-// out[t] = sum_j weights[t][j] * expert_out[t * top + j] (+ shared[t]), in the order of j.
-template <typename T>
-__global__ void moe_combine_kernel(const float* expert_out, const float* weights, const T* shared, int top, int width, T* out) {
+// out[t] = sum_j weights[t][j] * expert_out[t * top + j] (+ shared[t]), in the order of j. IDENTITY: a choice whose id is at or
+// past `experts` is an identity expert, whose output is h[t]. With `gate` (rows `gate_ld` apart) the shared expert's output is
+// multiplied by sigmoid(gate[t]).
+template <typename T, bool IDENTITY>
+__global__ void moe_combine_kernel(const float* expert_out, const float* weights, const T* shared, const int* ids, int experts, const T* h,
+                                   const float* gate, int gate_ld, int top, int width, T* out) {
   wait_for_predecessor();
   let_successor_start();
   const int t = blockIdx.x;
+  const float share = gate ? sigmoid_f(gate[static_cast<int64_t>(t) * gate_ld]) : 1.f;
   for (int d = threadIdx.x; d < width; d += blockDim.x) {
     float acc = 0.f;
-    for (int j = 0; j < top; ++j)
-      acc = fmaf(weights[static_cast<int64_t>(t) * top + j], expert_out[(static_cast<int64_t>(t) * top + j) * width + d], acc);
-    if (shared) acc += to_f32<T>(shared[static_cast<int64_t>(t) * width + d]);
+    const float own = IDENTITY ? to_f32<T>(h[static_cast<int64_t>(t) * width + d]) : 0.f;
+    for (int j = 0; j < top; ++j) {
+      const int64_t slot = static_cast<int64_t>(t) * top + j;
+      const float y = IDENTITY && ids[slot] >= experts ? own : expert_out[slot * width + d];
+      acc = fmaf(weights[slot], y, acc);
+    }
+    if (shared) acc = fmaf(share, to_f32<T>(shared[static_cast<int64_t>(t) * width + d]), acc);
     out[static_cast<int64_t>(t) * width + d] = from_f32<T>(acc);
+  }
+}
+
+// z <- max(z, 0)^2 in place, the activation of an ungated unit; packs of eight bfloat16 where alignment allows.
+template <typename T>
+__global__ void squared_relu_kernel(T* z, int64_t count) {
+  wait_for_predecessor();
+  let_successor_start();
+  for (int64_t i = blockIdx.x * static_cast<int64_t>(blockDim.x) + threadIdx.x; i < count; i += static_cast<int64_t>(gridDim.x) * blockDim.x)
+    z[i] = from_f32<T>(squared_relu(to_f32<T>(z[i])));
+}
+__global__ void squared_relu_wide_kernel(__nv_bfloat16* z, int64_t packs) {
+  wait_for_predecessor();
+  let_successor_start();
+  for (int64_t i = blockIdx.x * static_cast<int64_t>(blockDim.x) + threadIdx.x; i < packs; i += static_cast<int64_t>(gridDim.x) * blockDim.x) {
+    uint4 raw = reinterpret_cast<uint4*>(z)[i];
+    __nv_bfloat162* pair = reinterpret_cast<__nv_bfloat162*>(&raw);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const float2 u = __bfloat1622float2(pair[j]);
+      pair[j] = __floats2bfloat162_rn(squared_relu(u.x), squared_relu(u.y));
+    }
+    reinterpret_cast<uint4*>(z)[i] = raw;
   }
 }
 
@@ -528,16 +592,17 @@ __global__ void clamped_glu_wide_kernel(const __nv_bfloat16* gate_up, int64_t ro
 
 B200_API int b200_moe_tile_rows() { return kTileM; }
 
-B200_API int b200_moe_route(const float* z, const float* bias, int softmax_chosen, int tokens, int experts, int groups, int keep, int top,
+B200_API int b200_moe_route(const float* z, int ld, const float* bias, int rule, int tokens, int experts, int groups, int keep, int top,
                             float scale, int* ids, float* weights, cudaStream_t stream) {
   if (tokens == 0) return 0;
+  B200_REQUIRE(ld >= experts && rule >= ROUTE_SIGMOID && rule <= ROUTE_SOFTMAX_ALL, "moe_route: bad logits or rule");
   B200_REQUIRE(tokens > 0 && experts > 0 && groups > 0 && experts % groups == 0 && keep > 0 && keep <= groups && top > 0 &&
                    top <= keep * (experts / groups),
                "moe_route: %d experts in %d groups, %d kept, %d chosen", experts, groups, keep, top);
   const int warps = 4;
-  const size_t smem = sizeof(float) * warps * (experts + groups);
+  const size_t smem = sizeof(float) * warps * ((rule == ROUTE_SOFTMAX_ALL ? 2 : 1) * experts + groups);
   B200_REQUIRE(smem <= 48 * 1024, "moe_route: %d experts do not fit shared memory", experts);
-  launch_kernel(moe_route_kernel, dim3((tokens + warps - 1) / warps), dim3(32 * warps), smem, stream, z, bias, softmax_chosen, tokens, experts,
+  launch_kernel(moe_route_kernel, dim3((tokens + warps - 1) / warps), dim3(32 * warps), smem, stream, z, ld, bias, rule, tokens, experts,
                 groups, keep, top, scale, ids, weights);
   return b200_check_launch("moe_route");
 }
@@ -564,17 +629,17 @@ B200_API int b200_moe_mma_supported(int width, int ff) { return width % 8 == 0 &
 // `tile_rows`: what `moe_sort` was given. kTileM: the plain kernels, or with `use_mma` (bfloat16, sizes that
 // `moe_mma_supported` takes) the tensor-core form; four times kTileM: the tensor-core form only.
 B200_API int b200_moe_gate_up(const void* h, const void* weight, const int* place_slot, const int* tile_expert, const int* num_tiles,
-                              int max_tiles, int tile_rows, int top, int width, int ff, float limit, void* act, int dtype, int use_mma,
+                              int max_tiles, int tile_rows, int top, int width, int ff, int mats, float limit, void* act, int dtype, int use_mma,
                               cudaStream_t stream) {
   if (max_tiles == 0) return 0;
-  B200_REQUIRE(max_tiles > 0 && top > 0 && width > 0 && ff > 0 && limit >= 0.f, "moe_gate_up: bad sizes");
+  B200_REQUIRE(max_tiles > 0 && top > 0 && width > 0 && ff > 0 && limit >= 0.f && (mats == 1 || mats == 2), "moe_gate_up: bad sizes");
   const bool mma = dtype == DTYPE_BF16 && use_mma && b200_moe_mma_supported(width, ff) && aligned16(h) && aligned16(weight) && aligned16(act);
   B200_REQUIRE(tile_rows == kTileM || (mma && tile_rows == kTileM * kWideTiles), "moe_gate_up: tiles of %d rows are not taken here", tile_rows);
   const dim3 grid(max_tiles, (ff + kTileN - 1) / kTileN);
   B200_REQUIRE(grid.y <= 65535, "moe_gate_up: too many columns");
   if (dtype == DTYPE_F32) {
     launch_kernel(moe_gate_up_kernel<float>, grid, dim3(kGemmThreads), 0, stream, static_cast<const float*>(h),
-                  static_cast<const float*>(weight), place_slot, tile_expert, num_tiles, top, width, ff, limit, static_cast<float*>(act));
+                  static_cast<const float*>(weight), place_slot, tile_expert, num_tiles, top, width, ff, mats, limit, static_cast<float*>(act));
   } else if (mma) {
     const dim3 mma_grid(max_tiles, (ff + kMmaN - 1) / kMmaN);
     auto launch = [&](auto kernel, int threads, size_t smem) {
@@ -582,11 +647,16 @@ B200_API int b200_moe_gate_up(const void* h, const void* weight, const int* plac
       launch_kernel(kernel, mma_grid, dim3(threads), smem, stream, static_cast<const __nv_bfloat16*>(h), static_cast<const __nv_bfloat16*>(weight),
                     place_slot, tile_expert, num_tiles, top, width, ff, limit, static_cast<__nv_bfloat16*>(act));
     };
-    if (tile_rows == kTileM) launch(moe_gate_up_mma_kernel<1>, MmaShape<1>::threads, MmaShape<1>::smem(2));
-    else launch(moe_gate_up_mma_kernel<kWideTiles>, MmaShape<kWideTiles>::threads, MmaShape<kWideTiles>::smem(2));
+    if (tile_rows == kTileM) {
+      if (mats == 2) launch(moe_gate_up_mma_kernel<1, 2>, MmaShape<1>::threads, MmaShape<1>::smem(2));
+      else launch(moe_gate_up_mma_kernel<1, 1>, MmaShape<1>::threads, MmaShape<1>::smem(1));
+    } else {
+      if (mats == 2) launch(moe_gate_up_mma_kernel<kWideTiles, 2>, MmaShape<kWideTiles>::threads, MmaShape<kWideTiles>::smem(2));
+      else launch(moe_gate_up_mma_kernel<kWideTiles, 1>, MmaShape<kWideTiles>::threads, MmaShape<kWideTiles>::smem(1));
+    }
   } else if (dtype == DTYPE_BF16) {
     launch_kernel(moe_gate_up_kernel<__nv_bfloat16>, grid, dim3(kGemmThreads), 0, stream, static_cast<const __nv_bfloat16*>(h),
-                  static_cast<const __nv_bfloat16*>(weight), place_slot, tile_expert, num_tiles, top, width, ff, limit,
+                  static_cast<const __nv_bfloat16*>(weight), place_slot, tile_expert, num_tiles, top, width, ff, mats, limit,
                   static_cast<__nv_bfloat16*>(act));
   } else {
     return b200_fail("moe_gate_up: unknown dtype %d", dtype);
@@ -623,21 +693,47 @@ B200_API int b200_moe_down(const void* act, const void* weight, const int* place
   return b200_check_launch("moe_down");
 }
 
-B200_API int b200_moe_combine(const float* expert_out, const float* weights, const void* shared, int tokens, int top, int width, void* out,
-                              int dtype, cudaStream_t stream) {
+// `ids` null: no identity experts. `gate` null: the shared expert's output is added as it is.
+B200_API int b200_moe_combine(const float* expert_out, const float* weights, const void* shared, const int* ids, int experts, const void* h,
+                              const float* gate, int gate_ld, int tokens, int top, int width, void* out, int dtype, cudaStream_t stream) {
   if (tokens == 0) return 0;
-  B200_REQUIRE(tokens > 0 && top > 0 && width > 0, "moe_combine: bad sizes");
+  B200_REQUIRE(tokens > 0 && top > 0 && width > 0 && (ids == nullptr || h != nullptr), "moe_combine: bad sizes");
   const int threads = width >= 1024 ? 256 : 128;
+  auto launch = [&](auto kernel, auto* typed) {
+    using T = std::remove_pointer_t<decltype(typed)>;
+    launch_kernel(kernel, dim3(tokens), dim3(threads), 0, stream, expert_out, weights, static_cast<const T*>(shared), ids, experts,
+                  static_cast<const T*>(h), gate, gate_ld, top, width, typed);
+  };
   if (dtype == DTYPE_F32) {
-    launch_kernel(moe_combine_kernel<float>, dim3(tokens), dim3(threads), 0, stream, expert_out, weights, static_cast<const float*>(shared),
-                  top, width, static_cast<float*>(out));
+    if (ids) launch(moe_combine_kernel<float, true>, static_cast<float*>(out));
+    else launch(moe_combine_kernel<float, false>, static_cast<float*>(out));
   } else if (dtype == DTYPE_BF16) {
-    launch_kernel(moe_combine_kernel<__nv_bfloat16>, dim3(tokens), dim3(threads), 0, stream, expert_out, weights,
-                  static_cast<const __nv_bfloat16*>(shared), top, width, static_cast<__nv_bfloat16*>(out));
+    if (ids) launch(moe_combine_kernel<__nv_bfloat16, true>, static_cast<__nv_bfloat16*>(out));
+    else launch(moe_combine_kernel<__nv_bfloat16, false>, static_cast<__nv_bfloat16*>(out));
   } else {
     return b200_fail("moe_combine: unknown dtype %d", dtype);
   }
   return b200_check_launch("moe_combine");
+}
+
+B200_API int b200_squared_relu(void* z, int64_t count, int dtype, cudaStream_t stream) {
+  if (count == 0) return 0;
+  B200_REQUIRE(count > 0, "squared_relu: bad size");
+  const int threads = 256;
+  auto blocks = [&](int64_t items) {
+    const int64_t want = (items + threads - 1) / threads;
+    return dim3(static_cast<unsigned>(want < 65535 ? want : 65535));
+  };
+  if (dtype == DTYPE_F32) {
+    launch_kernel(squared_relu_kernel<float>, blocks(count), dim3(threads), 0, stream, static_cast<float*>(z), count);
+  } else if (dtype == DTYPE_BF16 && count % 8 == 0 && aligned16(z)) {
+    launch_kernel(squared_relu_wide_kernel, blocks(count / 8), dim3(threads), 0, stream, static_cast<__nv_bfloat16*>(z), count / 8);
+  } else if (dtype == DTYPE_BF16) {
+    launch_kernel(squared_relu_kernel<__nv_bfloat16>, blocks(count), dim3(threads), 0, stream, static_cast<__nv_bfloat16*>(z), count);
+  } else {
+    return b200_fail("squared_relu: unknown dtype %d", dtype);
+  }
+  return b200_check_launch("squared_relu");
 }
 
 B200_API int b200_clamped_glu(const void* gate_up, int rows, int ff, float limit, void* out, int dtype, cudaStream_t stream) {

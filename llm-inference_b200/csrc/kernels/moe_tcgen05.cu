@@ -7,7 +7,8 @@
 // the sorted activations, both K-major with 128-byte swizzle), one elected thread of a warp issues the
 // products, four warps read the accumulators back with `tcgen05.ld` and write the result. With two
 // matrices (gate and up) the block keeps two accumulators over the same X tile and its epilogue is the
-// clamped gated activation; with one (down) it stores 32-bit rows by slot. The gate/up product reads
+// clamped gated activation; with one (down) it stores 32-bit rows by slot, or (the up matrix of ungated experts) the
+// squared relu by place. The gate/up product reads
 // rows gathered into sorted order by `moe_gather_rows` in front (TMA does not gather rows); the down
 // product reads the activations where the first product wrote them. Places of padding hold whatever
 // the buffer held: a place is a column of D, so it harms no other place, and it is never stored.
@@ -121,7 +122,7 @@ struct ExpertProduct {
   void* out;            // MATS = 2: bfloat16 [places][n_total]; MATS = 1: float [slots][n_total]
 };
 
-template <int MATS>
+template <int MATS, bool SQUARED_RELU = false>
 __global__ void __launch_bounds__(kThreads)
 moe_tcgen05_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_constant__ CUtensorMap x_map, const ExpertProduct p) {
   extern __shared__ __align__(1024) unsigned char smem_raw[];
@@ -237,6 +238,9 @@ moe_tcgen05_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_const
             if (MATS == 2)
               static_cast<__nv_bfloat16*>(p.out)[static_cast<int64_t>(x_row + c0 + i) * p.n_total + n] =
                   __float2bfloat16_rn(clamped_glu(first[i], second[i], p.limit));
+            else if (SQUARED_RELU)
+              static_cast<__nv_bfloat16*>(p.out)[static_cast<int64_t>(x_row + c0 + i) * p.n_total + n] =
+                  __float2bfloat16_rn(fmaxf(first[i], 0.f) * fmaxf(first[i], 0.f));
             else
               static_cast<float*>(p.out)[static_cast<int64_t>(slot) * p.n_total + n] = first[i];
           }
@@ -299,10 +303,10 @@ int make_map(CUtensorMap* map, const void* base, int64_t rows, int K) {
   return 0;
 }
 
-template <int MATS>
+template <int MATS, bool SQUARED_RELU = false>
 int launch_product(const CUtensorMap& w_map, const CUtensorMap& x_map, const ExpertProduct& p, int max_tiles, cudaStream_t stream) {
   const size_t smem = static_cast<size_t>(p.stages) * (MATS + 1) * kTileBytes + 1024;
-  if (cudaFuncSetAttribute(moe_tcgen05_kernel<MATS>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)) != cudaSuccess)
+  if (cudaFuncSetAttribute(moe_tcgen05_kernel<MATS, SQUARED_RELU>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem)) != cudaSuccess)
     return b200_fail("moe_tcgen05: cannot size shared memory (%zu bytes)", smem);
   cudaLaunchConfig_t config = {};
   config.gridDim = dim3((p.n_total + kBlockRows - 1) / kBlockRows, max_tiles);
@@ -314,7 +318,7 @@ int launch_product(const CUtensorMap& w_map, const CUtensorMap& x_map, const Exp
   attribute[0].val.programmaticStreamSerializationAllowed = 1;
   config.attrs = attribute;
   config.numAttrs = b200_overlap_enabled() ? 1 : 0;
-  const cudaError_t status = cudaLaunchKernelEx(&config, moe_tcgen05_kernel<MATS>, w_map, x_map, p);
+  const cudaError_t status = cudaLaunchKernelEx(&config, moe_tcgen05_kernel<MATS, SQUARED_RELU>, w_map, x_map, p);
   if (status != cudaSuccess) return b200_fail("moe_tcgen05: %s", cudaGetErrorString(status));
   return 0;
 }
@@ -338,10 +342,11 @@ B200_API int b200_moe_gather_rows(const void* rows, const int* place_slot, int p
 
 // One of the two products over tiles of 128 sorted places. `weight`: the experts' matrices stacked, [experts * rows_per_expert][K];
 // `x`: [capacity][K] rows in sorted order. mats = 2: rows n and second_offset + n of an expert are gate and up of output column n,
-// `out` is bfloat16 [capacity][n_total] (the clamped gated activation); mats = 1: `out` is float [slots][n_total].
+// `out` is bfloat16 [capacity][n_total] (the clamped gated activation); mats = 1: `out` is float [slots][n_total], or, with
+// `squared_relu`, bfloat16 [capacity][n_total] (max(y, 0)^2).
 B200_API int b200_moe_product_tcgen05(const void* weight, const void* x, const int* place_slot, const int* tile_expert, const int* num_tiles,
                                       int max_tiles, int experts, int rows_per_expert, int second_offset, int n_total, int K, int mats,
-                                      float limit, void* out, int stages, int* err, cudaStream_t stream) {
+                                      int squared_relu, float limit, void* out, int stages, int* err, cudaStream_t stream) {
   if (max_tiles == 0) return 0;
   B200_REQUIRE(max_tiles > 0 && max_tiles <= 65535 && experts > 0 && rows_per_expert > 0 && n_total > 0 && K > 0 && K % 8 == 0 && (mats == 1 || mats == 2),
                "moe_product_tcgen05: bad sizes");
@@ -368,5 +373,6 @@ B200_API int b200_moe_product_tcgen05(const void* weight, const void* x, const i
   p.n_total = n_total;
   p.limit = limit;
   p.out = out;
+  if (mats == 1 && squared_relu) return launch_product<1, true>(w_map, x_map, p, max_tiles, stream);
   return mats == 2 ? launch_product<2>(w_map, x_map, p, max_tiles, stream) : launch_product<1>(w_map, x_map, p, max_tiles, stream);
 }

@@ -54,13 +54,14 @@ _SIGNATURES: dict[str, list] = {
     "b200_rope_kv_write": [c_void_p] * 7 + [c_int, c_int] + [c_void_p] * 3 + [c_int] * 8 + [c_void_p, c_void_p],
     "b200_paged_attention_plain": [c_void_p] * 6
     + [c_int, c_int, c_void_p]
-    + [c_int] * 6
-    + [c_float, c_int, c_float, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p],
+    + [c_int] * 7
+    + [c_float, c_int, c_float, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p],
     "b200_gemm_f32": [c_void_p] * 4 + [c_int] * 6 + [c_void_p],
-    "b200_paged_flash_attention": [c_void_p] * 8 + [c_int] * 11 + [c_float, c_int, c_int, c_int, c_float, c_void_p, c_int, c_int,
+    "b200_paged_flash_attention": [c_void_p] * 8 + [c_int] * 12 + [c_float, c_int, c_int, c_int, c_float, c_void_p, c_int, c_int, c_void_p,
                                    c_void_p, c_void_p, c_void_p],
     "b200_paged_decode_attention_tma": [c_void_p] * 8 + [c_int] * 8 + [c_float, c_int, c_int, c_void_p, c_void_p, c_void_p],
-    "b200_flash_prefill_tcgen05": [c_void_p] * 8 + [c_int] * 11 + [c_float, c_int, c_float, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p],
+    "b200_flash_prefill_tcgen05": [c_void_p] * 8 + [c_int] * 12 + [c_float, c_int, c_float, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p,
+                                   c_void_p],
     "b200_skinny_gemm": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int64, c_void_p, c_int, c_void_p],
     "b200_stream_gemm": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
     "b200_skinny_gemm_fold": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int64, c_void_p, c_int,
@@ -97,13 +98,19 @@ _SIGNATURES: dict[str, list] = {
     "b200_norm_kv_write": [c_void_p, c_int] + [c_void_p] * 4 + [c_int, c_int] + [c_void_p] * 5 + [c_int] * 9 + [c_float, c_int, c_int,
                            c_void_p, c_void_p],
     "b200_head_gate": [c_void_p, c_void_p] + [c_int] * 6 + [c_void_p, c_int, c_void_p],
-    "b200_moe_route": [c_void_p, c_void_p] + [c_int] * 6 + [c_float, c_void_p, c_void_p, c_void_p],
+    "b200_moe_route": [c_void_p, c_int, c_void_p] + [c_int] * 6 + [c_float, c_void_p, c_void_p, c_void_p],
     "b200_moe_sort": [c_void_p, c_int, c_int, c_int, c_int] + [c_void_p] * 4,
-    "b200_moe_gate_up": [c_void_p] * 5 + [c_int] * 5 + [c_float, c_void_p, c_int, c_int, c_void_p],
+    "b200_moe_gate_up": [c_void_p] * 5 + [c_int] * 6 + [c_float, c_void_p, c_int, c_int, c_void_p],
     "b200_moe_down": [c_void_p] * 5 + [c_int] * 4 + [c_void_p, c_int, c_int, c_void_p],
     "b200_moe_gather_rows": [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p],
-    "b200_moe_product_tcgen05": [c_void_p] * 5 + [c_int] * 7 + [c_float, c_void_p, c_int, c_void_p, c_void_p],
-    "b200_moe_combine": [c_void_p] * 3 + [c_int] * 3 + [c_void_p, c_int, c_void_p],
+    "b200_moe_product_tcgen05": [c_void_p] * 5 + [c_int] * 8 + [c_float, c_void_p, c_int, c_void_p, c_void_p],
+    "b200_moe_combine": [c_void_p] * 4 + [c_int, c_void_p, c_void_p] + [c_int] * 4 + [c_void_p, c_int, c_void_p],
+    "b200_squared_relu": [c_void_p, c_int64, c_int, c_void_p],
+    "b200_sandwich_norm": [c_void_p] * 3 + [c_float, c_float, c_void_p, c_void_p, c_float, c_float, c_void_p, c_float, c_void_p, c_int, c_int,
+                           c_void_p, c_int] + [c_void_p] * 7 + [c_int, c_void_p],
+    "b200_shift_norm": [c_void_p] * 10 + [c_int, c_int, c_void_p, c_int, c_void_p],
+    "b200_mlstm": [c_void_p] + [c_int] * 7 + [c_void_p, c_void_p, c_float] + [c_void_p] * 3 + [c_int] * 6 + [c_void_p] * 9
+                  + [c_float, c_void_p, c_int, c_void_p],
     "b200_clamped_glu": [c_void_p, c_int, c_int, c_float, c_void_p, c_int, c_void_p],
     "b200_mingru": [c_void_p, c_int] + [c_void_p] * 4 + [c_int] * 4 + [c_void_p] * 3 + [c_int, c_void_p],
     "b200_delta_general_prepare": [c_void_p] + [c_int] * 5 + [c_void_p] * 3 + [c_int] * 3 + [c_void_p] * 6 + [c_int, c_void_p],

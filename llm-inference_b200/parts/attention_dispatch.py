@@ -33,6 +33,8 @@ def attend(
     """``shape``: a soft cap, a bias by distance and a chunk of visible keys (``ops.ScoreShape``); the plain kernel, the
     mma.sync kernels and the tcgen05 prefill kernel take it. So shaped prompt portions run on tcgen05 where its sizes hold
     (heads of 128) and the mma.sync prefill form otherwise, and decoded tokens with any shaping the cp.async split-key kernel.
+    The same holds for sigmoid weights (``shape.sigmoid_bias``) and for first keys kept in front of a window
+    (``cache.keep_first``), which those kernels take as forms of their own.
 
     ``value_head`` >= 0: every query head's weights are applied to the values of that one kv head
     instead of its own (a mixer that mixes weights over heads asks for one such pass per kv head); the
@@ -42,6 +44,7 @@ def attend(
     tuned = (
         choice != "plain"
         and q.dtype == torch.bfloat16
+        and shape.tensor_cores_take(cache)
         and ops.flash_attention_supported(ctx, q_heads, kv_heads, head_dim, cache.page_size, decode=False)
     )
     if not tuned:
@@ -53,10 +56,10 @@ def attend(
     if decode_seqs and not ops.flash_attention_supported(ctx, q_heads, kv_heads, head_dim, cache.page_size, decode=True):
         decode_seqs = 0  # more than 16 query heads per kv head: the prefill form handles one-token runs too
     if decode_seqs:
-        reach = ctx.max_kv_len if not cache.window else min(ctx.max_kv_len, cache.window + 64)
+        reach = ctx.max_kv_len if not cache.window else min(ctx.max_kv_len, cache.window + 64 + cache.keep_first)
         if shape.chunk:
             reach = min(reach, shape.chunk)  # a decoded token sees its own chunk at most
-        tma = value_head < 0 and not shape and ops.decode_uses_tma(ctx, decode_seqs, q_heads, kv_heads, head_dim, cache.page_size)
+        tma = value_head < 0 and not shape and not cache.keep_first and ops.decode_uses_tma(ctx, decode_seqs, q_heads, kv_heads, head_dim, cache.page_size)
         splits = int(ctx.options.get("decode_splits", 0)) or ops.decode_splits(decode_seqs, kv_heads, reach, tma, ops.sm_count(ctx))
         ops.paged_flash_attention(
             ctx, cache, q, out, q_heads, kv_heads, head_dim, scale,

@@ -44,12 +44,14 @@ from ..weights.loader import TensorSpec
 class KVCacheSpec:
     """Paged keys and values: ``window`` 0 keeps every position, else the last ``window``.
     ``planes`` 1 keeps one row per token instead of a key row and a value row (a mixer whose
-    values are read out of its key rows, such as attention over cached latents)."""
+    values are read out of its key rows, such as attention over cached latents). With a window the
+    first ``keep_first`` positions of a request stay visible (and cached) too."""
 
     kv_heads: int
     head_dim: int
     window: int = 0
     planes: int = 2
+    keep_first: int = 0
 
 
 @dataclass(frozen=True)

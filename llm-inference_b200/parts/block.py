@@ -5,7 +5,7 @@ from __future__ import annotations
 import torch
 
 from . import ops
-from .base import Part, PartSpec, build_part, register_part
+from .base import CacheSpecs, Part, PartSpec, StateSpec, build_part, register_part
 from .context import CacheView, StepContext
 
 
@@ -189,6 +189,69 @@ class ParallelResidualBlock(Part):
         return ops.BranchSum(a, b)
 
 
+class SandwichResidualBlock(Part):
+    """``x += mult * norm1b(mixer(norm1(x))); x += mult * norm2b(feed_forward(norm2(x)))``: a norm on either side of each
+    sublayer (``feed_forward`` may be None). With ``shift`` (a tensor of factors per column) the mixer reads, instead of
+    ``h_t = norm1(x)_t``, the blend ``h_t + (h_(t-1) - h_t) * shift`` with the previous token's ``h`` (zeros in front of a
+    request's first token); a request's last ``h`` is part of its state.
+
+    A sublayer's output travels on as :class:`ops.NormedBranch`: the kernel of the norm that follows (this layer's second,
+    the next layer's first, or the model's last) also norms and adds it, so everything between two sublayers is one
+    kernel. The norms are norms of one group (``grouped_rmsnorm``)."""
+
+    def __init__(self, *, mixer: PartSpec, feed_forward: PartSpec | None, mixer_norm: PartSpec, mixer_out_norm: PartSpec,
+                 feed_forward_norm: PartSpec | None, feed_forward_out_norm: PartSpec | None, hidden_size: int, mult: float = 1.0,
+                 shift: str | None = None, unused: tuple[str, ...] = ()) -> None:
+        self.hidden_size, self.mult, self.shift_name, self.unused_names = hidden_size, float(mult), shift, tuple(unused)
+        self.mixer_norm, self.mixer_out_norm = build_part("norm", mixer_norm), build_part("norm", mixer_out_norm)
+        self.mixer = build_part("mixer", mixer)
+        self.feed_forward = build_part("feed_forward", feed_forward) if feed_forward is not None else None
+        second = (feed_forward_norm, feed_forward_out_norm) if feed_forward is not None else (None, None)
+        self.feed_forward_norm, self.feed_forward_out_norm = (build_part("norm", n) if n is not None else None for n in second)
+        self.parts = tuple(p for p in (self.mixer_norm, self.mixer_out_norm, self.mixer, self.feed_forward, self.feed_forward_norm,
+                                       self.feed_forward_out_norm) if p is not None)
+        self.graph_safe = all(p.graph_safe for p in self.parts)
+        self.factors: torch.Tensor | None = None
+
+    def tensor_specs(self):
+        from ..weights.loader import TensorSpec
+
+        specs = [spec for part in self.parts for spec in part.tensor_specs()]
+        if self.shift_name:
+            specs.append(TensorSpec(self.shift_name, (self.hidden_size,), init="half_plus_normal"))
+        # norms of a sublayer that the layer does not have may be in the checkpoint; they are read past
+        return specs + [TensorSpec(name, (self.hidden_size,), optional=True) for name in self.unused_names]
+
+    def load(self, tensors, dtype, device) -> None:
+        for part in self.parts:
+            part.load(tensors, dtype, device)
+        if self.shift_name:
+            self.factors = tensors[self.shift_name].to(device=device, dtype=torch.float32).contiguous()
+
+    def weight_bytes(self) -> int:
+        return sum(part.weight_bytes() for part in self.parts)
+
+    def cache_spec(self):
+        if not self.shift_name:
+            return self.mixer.cache_spec()
+        return CacheSpecs((self.mixer.cache_spec(), StateSpec(((self.hidden_size,),), (torch.float32,))))
+
+    def forward(self, ctx: StepContext, cache: CacheView | None, x: torch.Tensor, delta):
+        shift = None
+        if self.shift_name:
+            cache, slots = cache.members
+            shift = ops.TokenShift(self.factors, slots.state[0])
+        h = self.mixer_norm.forward(ctx, x, delta, shift=shift)
+        branch = self.mixer.forward(ctx, cache, h)
+        pending = ops.NormedBranch(branch, self.mixer_out_norm.weight, self.mult, self.mixer_out_norm.eps)
+        if self.feed_forward is None:
+            return pending
+        h = self.feed_forward_norm.forward(ctx, x, pending)
+        branch = self.feed_forward.forward(ctx, h)
+        return ops.NormedBranch(branch, self.feed_forward_out_norm.weight, self.mult, self.feed_forward_out_norm.eps)
+
+
+register_part("block", "sandwich_residual", SandwichResidualBlock)
 register_part("block", "parallel_residual", ParallelResidualBlock)
 register_part("block", "pre_norm_residual", PreNormResidualBlock)
 register_part("block", "post_norm_residual", PostNormResidualBlock)

@@ -57,6 +57,7 @@ class CacheView:
     max_pages: int = 0
     page_size: int = 0
     window: int = 0
+    keep_first: int = 0  # with a window: the first this many positions stay visible too
     state: list[torch.Tensor] | None = None
     members: list | None = None
 

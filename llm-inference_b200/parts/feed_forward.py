@@ -123,24 +123,38 @@ class RoutedExperts(Part):
 
     ``router="softmax_chosen"`` is another router: the ``top`` largest logits ``W_router h`` (+ ``router.b`` with
     ``router_bias``) are chosen and weighted by the softmax over the chosen logits alone (times ``route_scale``); it has no
-    groups. A ``limit`` of zero makes an expert ``W_down (silu(W_gate h) * (W_up h))``, without clamps. ``out_name`` is the
+    groups. ``router="softmax_all"`` is a third: scores are the softmax over all experts, ``correction`` (with ``router_bias``) is
+    added to the scores that compete only, a group counts by the largest of them, and a chosen expert's weight is its score
+    (times ``route_scale``), not renormalised. A ``limit`` of zero makes an expert ``W_down (silu(W_gate h) * (W_up h))``, without clamps. ``out_name`` is the
     buffer the result goes to (a layer that runs its feed-forward beside its mixer gives it one of its own).
+
+    ``activation="squared_relu"``: experts (and the shared one) are ungated, ``W_down max(W_up h, 0)^2``. The last ``identity``
+    of the ``experts + identity`` the router chooses from are identity experts: their output is ``h``. ``shared_gate``: the
+    shared expert's output is multiplied by ``sigmoid(W_sg h)``, one number per token; its row is one more of the router's
+    product.
 
     The experts' matrices are stacked (``[experts, 2 ff, hidden]`` with the gate rows first, and
     ``[experts, hidden, ff]``); a step sorts its (token, choice) pairs by expert and the two products
     walk the sorted runs, so only chosen experts' weights are read. Tensor names: ``prefix + router |
-    e<j>.{gate,up,down} | shared.{gate,up,down}``."""
+    router.b (or correction) | e<j>.{gate,up,down} | shared.{gate,up,down,sg}``."""
 
     def __init__(self, *, prefix: str, hidden_size: int, experts: int, top: int, intermediate_size: int, limit: float,
                  route_scale: float = 1.0, group_count: int = 1, group_keep: int = 1, shared_size: int | None = None,
                  shared_limit: float | None = None, router: str = "sigmoid_groups", router_bias: bool = False,
-                 out_name: str = "branch") -> None:
-        if router not in ("sigmoid_groups", "softmax_chosen"):
-            raise ValueError(f"router={router!r} must be 'sigmoid_groups' or 'softmax_chosen'")
+                 out_name: str = "branch", activation: str = "gated", identity: int = 0, shared_gate: bool = False) -> None:
+        if router not in ("sigmoid_groups", "softmax_chosen", "softmax_all"):
+            raise ValueError(f"router={router!r} must be 'sigmoid_groups', 'softmax_chosen' or 'softmax_all'")
+        if activation not in ("gated", "squared_relu"):
+            raise ValueError(f"activation={activation!r} must be 'gated' or 'squared_relu'")
+        if shared_gate and not shared_size:
+            raise ValueError("a gate on the shared expert wants a shared expert")
         if router == "softmax_chosen" and (group_count != 1 or group_keep != 1):
             raise ValueError("the router that weighs by a softmax over the chosen logits has no groups")
         self.prefix, self.hidden_size = prefix, hidden_size
         self.router, self.router_bias, self.out_name = router, bool(router_bias), out_name
+        self.bias_name = "correction" if router == "softmax_all" else "router.b"
+        self.gated, self.identity, self.shared_gate = activation == "gated", int(identity), bool(shared_gate)
+        self.choices = int(experts) + self.identity  # what the router chooses from
         self.b_router = None
         self.experts, self.top, self.intermediate_size, self.limit = int(experts), int(top), int(intermediate_size), float(limit)
         self.route_scale, self.group_count, self.group_keep = float(route_scale), int(group_count), int(group_keep)
@@ -150,14 +164,20 @@ class RoutedExperts(Part):
 
     def tensor_specs(self) -> list[TensorSpec]:
         p, h, i = self.prefix, self.hidden_size, self.intermediate_size
-        specs = [TensorSpec(p + "router", (self.experts, h))]
+        specs = [TensorSpec(p + "router", (self.choices, h))]
         if self.router_bias:
-            specs.append(TensorSpec(p + "router.b", (self.experts,)))
+            specs.append(TensorSpec(p + self.bias_name, (self.choices,)))
+
+        def unit(name: str, size: int) -> list[TensorSpec]:
+            front = ("gate", "up") if self.gated else ("up",)
+            return [TensorSpec(f"{p}{name}.{part}", (size, h)) for part in front] + [TensorSpec(f"{p}{name}.down", (h, size))]
+
         for e in range(self.experts):
-            specs += [TensorSpec(f"{p}e{e}.gate", (i, h)), TensorSpec(f"{p}e{e}.up", (i, h)), TensorSpec(f"{p}e{e}.down", (h, i))]
+            specs += unit(f"e{e}", i)
         if self.shared_size:
-            s = self.shared_size
-            specs += [TensorSpec(p + "shared.gate", (s, h)), TensorSpec(p + "shared.up", (s, h)), TensorSpec(p + "shared.down", (h, s))]
+            specs += unit("shared", self.shared_size)
+        if self.shared_gate:
+            specs.append(TensorSpec(p + "shared.sg", (1, h)))
         return specs
 
     def load(self, tensors, dtype, device) -> None:
@@ -166,13 +186,17 @@ class RoutedExperts(Part):
         def get(name: str) -> torch.Tensor:
             return tensors[p + name].to(device=device, dtype=dtype)
 
-        self.w_router = get("router").contiguous()
+        self.w_router = torch.cat([get("router"), get("shared.sg")]).contiguous() if self.shared_gate else get("router").contiguous()
         if self.router_bias:
-            self.b_router = tensors[p + "router.b"].to(device=device, dtype=torch.float32).contiguous()
-        self.w_gate_up = torch.stack([torch.cat([get(f"e{e}.gate"), get(f"e{e}.up")]) for e in range(self.experts)]).contiguous()
+            self.b_router = tensors[p + self.bias_name].to(device=device, dtype=torch.float32).contiguous()
+
+        def front(name: str) -> torch.Tensor:
+            return torch.cat([get(name + ".gate"), get(name + ".up")]) if self.gated else get(name + ".up")
+
+        self.w_gate_up = torch.stack([front(f"e{e}") for e in range(self.experts)]).contiguous()
         self.w_down = torch.stack([get(f"e{e}.down") for e in range(self.experts)]).contiguous()
         if self.shared_size:
-            self.w_shared_gate_up = torch.cat([get("shared.gate"), get("shared.up")]).contiguous()
+            self.w_shared_gate_up = front("shared").contiguous()
             self.w_shared_down = get("shared.down").contiguous()
 
     def weight_bytes(self) -> int:
@@ -183,25 +207,55 @@ class RoutedExperts(Part):
 
     def forward(self, ctx: StepContext, h: torch.Tensor) -> torch.Tensor:
         t, width = ctx.num_tokens, self.hidden_size
-        logits = ops.linear(ctx, h, self.w_router, ctx.buffer("moe_logits", (t, self.experts), torch.float32))
+        logits = ops.linear(ctx, h, self.w_router, ctx.buffer("moe_logits", (t, self.w_router.shape[0]), torch.float32))
         # Every routed layer keeps the step's choices in a buffer of its own, so that they can be read after
         # the step (expert load statistics, tests), also when the step was replayed from a captured graph.
         ids = ctx.buffer("moe_ids:" + self.prefix, (t, self.top), torch.int32)
         weights = ctx.buffer("moe_weights", (t, self.top), torch.float32)
-        ops.moe_route(ctx, logits, self.group_count, self.group_keep, self.top, self.route_scale, ids, weights, bias=self.b_router,
-                      softmax_chosen=self.router == "softmax_chosen")
+        ops.moe_route(ctx, logits[:, : self.choices], self.group_count, self.group_keep, self.top, self.route_scale, ids, weights, bias=self.b_router,
+                      softmax_chosen=self.router == "softmax_chosen", softmax_all=self.router == "softmax_all")
         expert_out = ops.moe_experts(
             ctx, h, ids, self.w_gate_up, self.w_down, self.limit, ctx.buffer("moe_expert_out", (t * self.top, width), torch.float32, per_token=False)
         )
         shared = None
         if self.shared_size:
-            gate_up = ops.linear(ctx, h, self.w_shared_gate_up, ctx.buffer("gate_up", (t, 2 * self.shared_size)))
-            act = ops.clamped_glu(ctx, gate_up, self.shared_limit, ctx.buffer("act", (t, self.shared_size)))
+            if self.gated:
+                gate_up = ops.linear(ctx, h, self.w_shared_gate_up, ctx.buffer("gate_up", (t, 2 * self.shared_size)))
+                act = ops.clamped_glu(ctx, gate_up, self.shared_limit, ctx.buffer("act", (t, self.shared_size)))
+            else:
+                act = ops.linear_squared_relu(ctx, h, self.w_shared_gate_up, ctx.buffer("act", (t, self.shared_size)))
             shared = ops.linear(ctx, act, self.w_shared_down, ctx.buffer("moe_shared", (t, width)))
-        return ops.moe_combine(ctx, expert_out, weights, shared, ctx.buffer(self.out_name, (t, width)))
+        return ops.moe_combine(
+            ctx, expert_out, weights, shared, ctx.buffer(self.out_name, (t, width)),
+            identity=(ids, self.experts, h) if self.identity else None, shared_gate=logits[:, self.choices] if self.shared_gate else None,
+        )
+
+
+class SquaredReLUFeedForward(Part):
+    """``down(max(up(h), 0)^2)`` without biases. Tensor names: ``prefix + up | down``."""
+
+    def __init__(self, *, prefix: str, hidden_size: int, intermediate_size: int) -> None:
+        self.prefix, self.hidden_size, self.intermediate_size = prefix, hidden_size, int(intermediate_size)
+        self.w_up = self.w_down = None
+
+    def tensor_specs(self) -> list[TensorSpec]:
+        p, h, i = self.prefix, self.hidden_size, self.intermediate_size
+        return [TensorSpec(p + "up", (i, h)), TensorSpec(p + "down", (h, i))]
+
+    def load(self, tensors, dtype, device) -> None:
+        self.w_up, self.w_down = (tensors[self.prefix + n].to(device=device, dtype=dtype).contiguous() for n in ("up", "down"))
+
+    def weight_bytes(self) -> int:
+        return (self.w_up.numel() + self.w_down.numel()) * self.w_down.element_size()
+
+    def forward(self, ctx: StepContext, h: torch.Tensor) -> torch.Tensor:
+        t = ctx.num_tokens
+        act = ops.linear_squared_relu(ctx, h, self.w_up, ctx.buffer("act", (t, self.intermediate_size)))
+        return ops.linear(ctx, act, self.w_down, ctx.buffer("branch", (t, self.hidden_size)))
 
 
 register_part("feed_forward", "swiglu", SwiGLU)
 register_part("feed_forward", "poly_norm", PolyNormFeedForward)
 register_part("feed_forward", "routed_experts", RoutedExperts)
 register_part("feed_forward", "clamped_glu", ClampedGLU)
+register_part("feed_forward", "squared_relu", SquaredReLUFeedForward)

@@ -12,13 +12,15 @@ from .context import CacheView, StepContext
 
 def padded_head_size(dim: int, vdim: int) -> int:
     """The row width of the cache: keys (``dim``) and values (``vdim``) share one arena shape, and the
-    tensor-core attention kernels take heads of 64 or 128; smaller heads are padded with zeros up to
+    tensor-core attention kernels take heads of 64, 128 or 192; smaller heads are padded with zeros up to
     those, larger ones to a multiple of 16."""
     need = max(dim, vdim)
     if need <= 64:
         return 64
     if need <= 128:
         return 128
+    if need <= 192:
+        return 192
     return (need + 15) // 16 * 16
 
 

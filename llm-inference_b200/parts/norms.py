@@ -62,7 +62,9 @@ class GroupedRMSNorm(Part):
     Two uses. As the norm of the stream itself (``forward``, the interface of every norm part; the
     model's last norm). And as the norm of a branch's *output* in a layer that adds
     ``mult * scale * norm(branch(x))`` to its stream (``add_branch``); the same kernel can then also
-    form the weighted average over depth that such a layer hands on (parts/block.py)."""
+    form the weighted average over depth that such a layer hands on (parts/block.py). With one group ``forward`` also
+    takes a sublayer's output that has a norm of its own and is still to be added (``ops.NormedBranch``) and a blend with
+    the previous token's row (``ops.TokenShift``)."""
 
     foldable = False
 
@@ -87,11 +89,14 @@ class GroupedRMSNorm(Part):
         return self.weight.numel() * 4
 
     def forward(self, ctx: StepContext, x: torch.Tensor, delta, rows: torch.Tensor | None = None, out_name: str = "normed",
-                folded_ok: bool = False) -> torch.Tensor:
-        if delta is not None:
-            raise ValueError("a grouped norm reads a stream that is up to date; it takes no pending branch output")
+                folded_ok: bool = False, shift: ops.TokenShift | None = None) -> torch.Tensor:
         count = x.shape[0] if rows is None else rows.shape[0]
         out = ctx.buffer(out_name, (count, self.hidden_size), per_token=rows is None)
+        if self.groups == 1 and (isinstance(delta, ops.NormedBranch) or shift is not None):
+            # a sublayer's output with a norm of its own still to be added: both norms and the add are one kernel
+            return ops.sandwich_norm(ctx, x, delta, self.weight, self.eps, out, rows, shift)
+        if delta is not None or shift is not None:
+            raise ValueError("a norm in groups reads a stream that is up to date; it takes no pending branch output")
         return ops.grouped_rmsnorm(ctx, x, self.weight, self.groups, self.eps, out, rows)
 
     def add_branch(self, ctx: StepContext, x_in: torch.Tensor, branch: torch.Tensor, scale: torch.Tensor | None, mult: float,

@@ -359,16 +359,25 @@ class ScoreShape:
     bias: torch.Tensor | None = None
     chunk: int = 0
     bias_peak: torch.Tensor | None = None  # float32 [q_heads]: each row's largest entry (the tcgen05 kernel bounds exponents with it)
+    sigmoid_bias: torch.Tensor | None = None  # float32 [q_heads]: a visible key weighs sigmoid(score + bias), nothing is normalised
 
     def __bool__(self) -> bool:
-        return bool(self.softcap > 0.0 or self.bias is not None or self.chunk > 0)
+        return bool(self.softcap > 0.0 or self.bias is not None or self.chunk > 0 or self.sigmoid_bias is not None)
+
+    def tensor_cores_take(self, cache: CacheView) -> bool:
+        """The tensor-core kernels have one form per kind of score: a cap, bias or chunk does not go together with sigmoid
+        weights or with first keys kept in front of a window (the plain kernel takes every combination)."""
+        changed = self.softcap > 0.0 or self.bias is not None or self.chunk > 0
+        return not (changed and (self.sigmoid_bias is not None or (cache.window and cache.keep_first)))
 
     def arguments(self, q_heads: int) -> list:
         if self.bias is not None:
             _need(self.bias.dtype == torch.float32 and self.bias.dim() == 2 and self.bias.shape[0] == q_heads and self.bias.is_contiguous(),
                   "attention: the bias by distance is float32 [q_heads, reach + 1]")
+        if self.sigmoid_bias is not None:
+            _need(self.sigmoid_bias.dtype == torch.float32 and self.sigmoid_bias.numel() == q_heads, "attention: the sigmoid's bias is float32 [q_heads]")
         reach = self.bias.shape[1] - 1 if self.bias is not None else 0
-        return [c_float(self.softcap), ptr(self.bias), c_int(reach), c_int(self.chunk)]
+        return [c_float(self.softcap), ptr(self.bias), c_int(reach), c_int(self.chunk), ptr(self.sigmoid_bias)]
 
 
 NO_SHAPE = ScoreShape()
@@ -405,7 +414,8 @@ def paged_attention_plain(
         ptr(cache.block_table), c_int(cache.max_pages), c_int(cache.num_pages),
         ptr(out) if first_token == 0 else _offset(out, first_token * row_bytes),
         c_int(tokens), c_int(q_heads), c_int(kv_heads), c_int(head_dim), c_int(cache.page_size),
-        c_int(cache.window), c_float(scale), c_int(value_head), *shape.arguments(q_heads), c_int(dtype_code(q.dtype)), ptr(ctx.err),
+        c_int(cache.window), c_int(cache.keep_first), c_float(scale), c_int(value_head), *shape.arguments(q_heads), c_int(dtype_code(q.dtype)),
+        ptr(ctx.err),
         ctx.stream,
     )
     return out
@@ -511,7 +521,7 @@ def paged_flash_attention(
     # slow to place. The TMA kernel always goes through scratch unless told otherwise: at
     # batch 1 both forms take 1.10 ms per step (the cp.async kernel 1.15), at batch 2 scratch
     # 1.10 and the cluster 1.12, from batch 4 on the cluster loses.
-    use_tma = decode and value_head == -1 and not shape and decode_uses_tma(ctx, num_seqs, q_heads, kv_heads, head_dim, cache.page_size)
+    use_tma = decode and value_head == -1 and not shape and not cache.keep_first and decode_uses_tma(ctx, num_seqs, q_heads, kv_heads, head_dim, cache.page_size)
     merge = ctx.options.get("attention_merge", "auto")
     if merge == "auto":
         merge = "cluster" if num_seqs * kv_heads * planes <= 4 and not use_tma else "scratch"
@@ -534,7 +544,7 @@ def paged_flash_attention(
         "b200_paged_flash_attention", ptr(q), ptr(cache.keys), ptr(cache.values), ptr(out), ptr(cache.block_table),
         ptr(ctx.seq_q_start), ptr(ctx.seq_q_len), ptr(ctx.seq_kv_len), c_int(first_seq), c_int(num_seqs),
         c_int(num_seqs if decode else ctx.num_tokens), c_int(max_q_len), c_int(cache.max_pages), c_int(cache.num_pages),
-        c_int(q_heads), c_int(kv_heads), c_int(head_dim), c_int(cache.page_size), c_int(cache.window), c_float(scale),
+        c_int(q_heads), c_int(kv_heads), c_int(head_dim), c_int(cache.page_size), c_int(cache.window), c_int(cache.keep_first), c_float(scale),
         c_int(1 if decode else 0), c_int(splits), c_int(value_head), *shape.arguments(q_heads), ptr(scratch), ptr(ctx.err), ctx.stream,
     )
     if scratch is not None:
@@ -576,8 +586,8 @@ def paged_prefill_attention_tcgen05(
         "b200_flash_prefill_tcgen05", ptr(q), ptr(cache.keys), ptr(cache.values), ptr(out), ptr(cache.block_table),
         ptr(ctx.seq_q_start), ptr(ctx.seq_q_len), ptr(ctx.seq_kv_len), c_int(first_seq), c_int(num_seqs), c_int(max_q_len),
         c_int(ctx.max_kv_len), c_int(cache.max_pages), c_int(cache.num_pages), c_int(q_heads), c_int(kv_heads),
-        c_int(head_dim), c_int(cache.page_size), c_int(cache.window), c_float(scale), c_int(value_head), c_float(shape.softcap), ptr(shape.bias), ptr(shape.bias_peak), reach,
-        c_int(shape.chunk), ptr(ctx.err), ctx.stream,
+        c_int(head_dim), c_int(cache.page_size), c_int(cache.window), c_int(cache.keep_first), c_float(scale), c_int(value_head), c_float(shape.softcap),
+        ptr(shape.bias), ptr(shape.bias_peak), reach, c_int(shape.chunk), ptr(shape.sigmoid_bias), ptr(ctx.err), ctx.stream,
     )
     return out
 
@@ -1029,17 +1039,20 @@ def head_gate(ctx: StepContext, attn: torch.Tensor, proj: torch.Tensor | None, g
 
 
 def moe_route(ctx: StepContext, logits: torch.Tensor, groups: int, keep: int, top: int, scale: float, ids: torch.Tensor, weights: torch.Tensor,
-              *, bias: torch.Tensor | None = None, softmax_chosen: bool = False) -> None:
+              *, bias: torch.Tensor | None = None, softmax_chosen: bool = False, softmax_all: bool = False) -> None:
     """``bias`` (float32 ``[experts]``) is added to the logits first. ``softmax_chosen``: an expert's score is its logit
-    and the chosen experts' weights are the softmax over their logits alone (times ``scale``); otherwise the score is
-    the logit's sigmoid and the weights are the chosen scores over their sum."""
+    and the chosen experts' weights are the softmax over their logits alone (times ``scale``). ``softmax_all``: its score
+    is the softmax over all experts; ``bias`` is then added to the scores that compete only, a group counts by its
+    largest, and a chosen expert's weight is its score times ``scale``. Otherwise the score is the logit's sigmoid and
+    the weights are the chosen scores over their sum. ``logits`` may be the leading columns of wider rows."""
     tokens, experts = logits.shape
+    rule = 2 if softmax_all else (1 if softmax_chosen else 0)
     _need(bias is None or (bias.dtype == torch.float32 and bias.numel() == experts and bias.is_contiguous()), "moe_route: the bias is float32 [experts]")
-    _need(logits.dtype == torch.float32 and logits.is_contiguous(), "moe_route: router logits are contiguous float32")
+    _need(logits.dtype == torch.float32 and logits.stride(1) == 1, "moe_route: router logits are float32 rows")
     _need(ids.dtype == torch.int32 and tuple(ids.shape) == (tokens, top) and ids.is_contiguous(), "moe_route: bad ids")
     _need(weights.dtype == torch.float32 and tuple(weights.shape) == (tokens, top) and weights.is_contiguous(), "moe_route: bad weights")
     ctx.lib.call(
-        "b200_moe_route", ptr(logits), ptr(bias), c_int(1 if softmax_chosen else 0), c_int(tokens), c_int(experts), c_int(groups), c_int(keep), c_int(top), c_float(scale), ptr(ids),
+        "b200_moe_route", ptr(logits), c_int(logits.stride(0)), ptr(bias), c_int(rule), c_int(tokens), c_int(experts), c_int(groups), c_int(keep), c_int(top), c_float(scale), ptr(ids),
         ptr(weights), ctx.stream,
     )
 
@@ -1052,16 +1065,18 @@ def moe_experts(
     ctx: StepContext, h: torch.Tensor, ids: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, limit: float, out: torch.Tensor
 ) -> torch.Tensor:
     """``out[t * top + j] = expert ids[t, j] applied to h[t]`` (float32, not yet weighted). ``w_gate_up`` is
-    ``[experts, 2 * ff, width]`` (gate rows, then up rows), ``w_down`` ``[experts, width, ff]``. The slots are sorted by
-    expert into runs of whole tiles, then the two products walk the tiles (tall tiles on tcgen05 read rows that a
+    ``[experts, 2 * ff, width]`` (gate rows, then up rows), or ``[experts, ff, width]`` for ungated experts (``max(up, 0)^2``);
+    ``w_down`` is ``[experts, width, ff]``. Ids at or past ``experts`` have no matrices: their rows of ``out`` are left as they
+    were. The slots are sorted by expert into runs of whole tiles, then the two products walk the tiles (tall tiles on tcgen05 read rows that a
     gather pass has put into sorted order)."""
     tokens, width = h.shape
     top = ids.shape[1]
     experts, twice, _ = w_gate_up.shape
-    ff = twice // 2
+    ff = w_down.shape[2]
+    mats = twice // ff
     slots = tokens * top
     _need(h.is_contiguous() and w_gate_up.is_contiguous() and w_down.is_contiguous() and w_gate_up.dtype == h.dtype and w_down.dtype == h.dtype, "moe_experts: bad operands")
-    _need(tuple(w_gate_up.shape) == (experts, 2 * ff, width) and tuple(w_down.shape) == (experts, width, ff), "moe_experts: bad weights")
+    _need(mats in (1, 2) and tuple(w_gate_up.shape) == (experts, mats * ff, width) and tuple(w_down.shape) == (experts, width, ff), "moe_experts: bad weights")
     _need(out.dtype == torch.float32 and tuple(out.shape) == (slots, width) and out.is_contiguous(), "moe_experts: bad output")
     # bfloat16 runs on tensor cores where the sizes allow, and a step with many slots per expert sorts them into tiles
     # four times as tall (128 places), which the tcgen05 form takes; short steps keep tiles of 32 and mma.sync.
@@ -1085,17 +1100,17 @@ def moe_experts(
         stages = c_int(int(ctx.options.get("moe_stages", 0)))
         ctx.lib.call(
             "b200_moe_product_tcgen05", ptr(w_gate_up), ptr(sorted_rows), ptr(place_slot), ptr(tile_expert), ptr(num_tiles), c_int(max_tiles),
-            c_int(experts), c_int(2 * ff), c_int(ff), c_int(ff), c_int(width), c_int(2), c_float(limit), ptr(act), stages, ptr(ctx.err), ctx.stream,
+            c_int(experts), c_int(mats * ff), c_int(ff), c_int(ff), c_int(width), c_int(mats), c_int(1 if mats == 1 else 0), c_float(limit), ptr(act), stages, ptr(ctx.err), ctx.stream,
         )
         ctx.lib.call(
             "b200_moe_product_tcgen05", ptr(w_down), ptr(act), ptr(place_slot), ptr(tile_expert), ptr(num_tiles), c_int(max_tiles),
-            c_int(experts), c_int(width), c_int(0), c_int(width), c_int(ff), c_int(1), c_float(limit), ptr(out), stages, ptr(ctx.err), ctx.stream,
+            c_int(experts), c_int(width), c_int(0), c_int(width), c_int(ff), c_int(1), c_int(0), c_float(limit), ptr(out), stages, ptr(ctx.err), ctx.stream,
         )
         return out
     code, use = c_int(dtype_code(h.dtype)), c_int(1 if tensor_cores else 0)
     ctx.lib.call(
         "b200_moe_gate_up", ptr(h), ptr(w_gate_up), ptr(place_slot), ptr(tile_expert), ptr(num_tiles), c_int(max_tiles), c_int(tile), c_int(top),
-        c_int(width), c_int(ff), c_float(limit), ptr(act), code, use, ctx.stream,
+        c_int(width), c_int(ff), c_int(mats), c_float(limit), ptr(act), code, use, ctx.stream,
     )
     ctx.lib.call(
         "b200_moe_down", ptr(act), ptr(w_down), ptr(place_slot), ptr(tile_expert), ptr(num_tiles), c_int(max_tiles), c_int(tile), c_int(width),
@@ -1104,13 +1119,21 @@ def moe_experts(
     return out
 
 
-def moe_combine(ctx: StepContext, expert_out: torch.Tensor, weights: torch.Tensor, shared: torch.Tensor | None, out: torch.Tensor) -> torch.Tensor:
+def moe_combine(ctx: StepContext, expert_out: torch.Tensor, weights: torch.Tensor, shared: torch.Tensor | None, out: torch.Tensor, *,
+                identity: tuple[torch.Tensor, int, torch.Tensor] | None = None, shared_gate: torch.Tensor | None = None) -> torch.Tensor:
+    """``out[t] = sum_j weights[t, j] * expert_out[t * top + j] (+ shared[t])``. ``identity = (ids, experts, h)``: a choice whose
+    id is at or past ``experts`` contributes ``h[t]`` instead. ``shared_gate`` (a float32 column, rows any stride apart): the
+    shared output is multiplied by its sigmoid."""
     tokens, top = weights.shape
+    ids, experts, h = identity if identity is not None else (None, 0, None)
+    _need(ids is None or (ids.dtype == torch.int32 and ids.shape == weights.shape and ids.is_contiguous() and h.shape == out.shape and h.dtype == out.dtype and h.is_contiguous()), "moe_combine: bad identity experts")
+    _need(shared_gate is None or (shared is not None and shared_gate.dtype == torch.float32 and shared_gate.shape[0] == tokens), "moe_combine: bad gate of the shared expert")
     width = out.shape[1]
     _need(expert_out.dtype == torch.float32 and tuple(expert_out.shape) == (tokens * top, width) and expert_out.is_contiguous(), "moe_combine: bad expert outputs")
     _need(out.is_contiguous() and out.shape[0] == tokens and (shared is None or (shared.shape == out.shape and shared.dtype == out.dtype and shared.is_contiguous())), "moe_combine: bad operands")
     ctx.lib.call(
-        "b200_moe_combine", ptr(expert_out), ptr(weights), ptr(shared), c_int(tokens), c_int(top), c_int(width), ptr(out),
+        "b200_moe_combine", ptr(expert_out), ptr(weights), ptr(shared), ptr(ids), c_int(experts), ptr(h), ptr(shared_gate),
+        c_int(shared_gate.stride(0) if shared_gate is not None else 0), c_int(tokens), c_int(top), c_int(width), ptr(out),
         c_int(dtype_code(out.dtype)), ctx.stream,
     )
     return out
@@ -1383,3 +1406,114 @@ def qk_norm_rope_write(
         c_int(dtype_code(proj.dtype)), ptr(ctx.err), ctx.stream,
     )
     return q_out
+
+
+# -- norms on either side of a sublayer, the previous token's row, the matrix memory, the squared relu -----------------
+
+
+@dataclass
+class ScaledPair:
+    """The outputs of two mixers that ran side by side, not yet combined: ``a_scale * a + b_scale * b (+ constant)`` with a
+    float32 constant per column (an output bias). The norm kernel that adds the branch to the stream combines them."""
+
+    a: torch.Tensor
+    b: torch.Tensor
+    a_scale: float
+    b_scale: float
+    constant: torch.Tensor | None = None
+
+
+@dataclass
+class NormedBranch:
+    """A sublayer's output (a tensor or a :class:`ScaledPair`) still to be normed and added: ``x += mult * weight * y / rms(y)``."""
+
+    branch: Any
+    weight: torch.Tensor
+    mult: float
+    eps: float
+
+
+@dataclass
+class TokenShift:
+    """What a blend with the previous token's row needs: the factors per column and the slots ``[slots, hidden]`` (float32)."""
+
+    factors: torch.Tensor
+    slots: torch.Tensor
+
+
+def sandwich_norm(ctx: StepContext, x: torch.Tensor, delta: NormedBranch | None, weight: torch.Tensor, eps: float, out: torch.Tensor,
+                  rows: torch.Tensor | None = None, shift: TokenShift | None = None) -> torch.Tensor:
+    """``x += delta`` (normed and scaled, see :class:`NormedBranch`; not written back when ``rows`` picks rows), ``out = weight
+    * x / rms(x)``; with ``shift`` then ``out[t] += (out[t - 1] - out[t]) * factors``, a request's first token of the step taking
+    its slot for ``out[t - 1]`` and its last one moving the slot on. One kernel; two when a step with a shift holds runs of
+    more than one token (a token's neighbour is then another block's row)."""
+    hidden = x.shape[1]
+    count = x.shape[0] if rows is None else rows.shape[0]
+    _need(x.dtype == torch.float32 and x.is_contiguous(), "sandwich_norm: the residual stream is contiguous float32")
+    _need(weight.dtype == torch.float32 and weight.numel() == hidden, "sandwich_norm: weight must be float32 [hidden]")
+    _need(tuple(out.shape) == (count, hidden) and out.is_contiguous(), "sandwich_norm: bad output shape")
+    branch = delta.branch if delta is not None else None
+    pair = branch if isinstance(branch, ScaledPair) else ScaledPair(branch, None, 1.0, 0.0)
+    for d in (pair.a, pair.b):
+        _need(d is None or (d.shape == x.shape and d.dtype == out.dtype and d.is_contiguous()), "sandwich_norm: bad branch output")
+    for c in (pair.constant, delta.weight if delta is not None else None):
+        _need(c is None or (c.dtype == torch.float32 and c.numel() == hidden), "sandwich_norm: constants are float32 [hidden]")
+    mode, rstd, previous = 0, None, None
+    if shift is not None:
+        _need(rows is None, "sandwich_norm: a blend with the previous token wants the whole step")
+        _need(shift.factors.dtype == torch.float32 and shift.factors.numel() == hidden, "sandwich_norm: blend factors are float32 [hidden]")
+        _need(shift.slots.dtype == torch.float32 and tuple(shift.slots.shape[1:]) == (hidden,) and shift.slots.is_contiguous(), "sandwich_norm: the slots are float32 [slots, hidden]")
+        mode = 1 if ctx.num_tokens == ctx.num_seqs else 2
+        if mode == 2:
+            rstd = ctx.buffer("shift_rstd", (count,), torch.float32)
+            previous = ctx.buffer("shift_previous", (ctx.num_seqs, hidden), torch.float32, per_token=False)
+    ctx.lib.call(
+        "b200_sandwich_norm", ptr(x), ptr(pair.a), ptr(pair.b), c_float(pair.a_scale), c_float(pair.b_scale), ptr(pair.constant),
+        ptr(delta.weight if delta is not None else None), c_float(delta.mult if delta is not None else 0.0),
+        c_float(delta.eps if delta is not None else 0.0), ptr(weight), c_float(eps), ptr(rows), c_int(count), c_int(hidden), ptr(out), c_int(mode),
+        ptr(shift.factors if shift is not None else None), ptr(shift.slots if shift is not None else None), ptr(ctx.token_seq),
+        ptr(ctx.seq_q_start), ptr(ctx.seq_slot), ptr(rstd), ptr(previous), c_int(dtype_code(out.dtype)), ctx.stream,
+    )
+    if mode == 2:
+        ctx.lib.call(
+            "b200_shift_norm", ptr(x), ptr(rstd), ptr(weight), ptr(shift.factors), ptr(previous), ptr(shift.slots), ptr(ctx.token_seq),
+            ptr(ctx.seq_q_start), ptr(ctx.seq_q_len), ptr(ctx.seq_slot), c_int(count), c_int(hidden), ptr(out), c_int(dtype_code(out.dtype)), ctx.stream,
+        )
+    return out
+
+
+def mlstm(ctx: StepContext, proj: torch.Tensor, columns: tuple[int, int, int, int, int, int], i_bias: torch.Tensor, f_bias: torch.Tensor, cap: float,
+          state: list[torch.Tensor], heads: int, dk: int, dv: int, norm: torch.Tensor, eps: float, out: torch.Tensor) -> torch.Tensor:
+    """The matrix memory between its projections and its output product (csrc/kernels/mlstm.cu). ``proj`` is float32;
+    ``columns`` says where q, k, v, the output gate's logits and the two gates' logits begin; ``state`` is ``[S, n, m]``
+    by slot."""
+    tokens = proj.shape[0]
+    S, n, m = state
+    f32 = torch.float32
+    _need(proj.dtype == f32 and proj.is_contiguous() and proj.shape[1] >= 2 * heads * (dk + dv + 1), "mlstm: the projections are float32 rows of q, k, v and the gates")
+    _need(S.dtype == f32 and tuple(S.shape[1:]) == (heads, dk, dv) and S.is_contiguous(), "mlstm: S is float32 [slots, heads, dk, dv]")
+    _need(n.dtype == f32 and tuple(n.shape[1:]) == (heads, dk) and n.is_contiguous() and m.dtype == f32 and tuple(m.shape[1:]) == (heads,) and m.is_contiguous(), "mlstm: n is float32 [slots, heads, dk], m float32 [slots, heads]")
+    _need(all(b.dtype == f32 and b.numel() == heads for b in (i_bias, f_bias)) and norm.dtype == f32 and norm.numel() == heads * dv, "mlstm: bad constants")
+    _need(tuple(out.shape) == (tokens, heads * dv) and out.is_contiguous(), "mlstm: bad output")
+    single = ctx.num_tokens == ctx.num_seqs
+    gates = [None] * 3 if single else [ctx.buffer("mlstm_" + name, (tokens, heads), f32) for name in ("keep", "put", "least")]
+    num, den = ctx.buffer("mlstm_num", (tokens, heads * dv), f32), ctx.buffer("mlstm_den", (tokens, heads), f32)
+    ctx.lib.call(
+        "b200_mlstm", ptr(proj), c_int(proj.shape[1]), *(c_int(c) for c in columns), ptr(i_bias), ptr(f_bias), c_float(cap), ptr(ctx.seq_q_start),
+        ptr(ctx.seq_q_len), ptr(ctx.seq_slot), c_int(ctx.num_seqs), c_int(tokens), c_int(1 if single else 0), c_int(heads), c_int(dk), c_int(dv),
+        ptr(S), ptr(n), ptr(m), *(ptr(g) for g in gates), ptr(num), ptr(den), ptr(norm), c_float(eps), ptr(out), c_int(dtype_code(out.dtype)), ctx.stream,
+    )
+    ctx.lib.calls += 1 if single else 2  # the recurrence and the output kernel (and the gates') are launches of their own
+    return out
+
+
+def linear_squared_relu(ctx: StepContext, x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+    """``out = max(x @ weight.T, 0)^2``."""
+    return squared_relu(ctx, linear(ctx, x, weight, out))
+
+
+def squared_relu(ctx: StepContext, z: torch.Tensor) -> torch.Tensor:
+    """``z <- max(z, 0)^2`` in place."""
+    _need(z.is_contiguous(), "squared_relu: a contiguous buffer")
+    ctx.lib.call("b200_squared_relu", ptr(z), c_int64(z.numel()), c_int(dtype_code(z.dtype)), ctx.stream)
+    return z

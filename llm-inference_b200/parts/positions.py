@@ -30,6 +30,10 @@ class RotaryEncoding(Part):
         # hi = min(ceil(t(slow)), rotary_dims - 1), frequency i is f / factor * r + f * (1 - r) with
         # r = clamp((i - lo) / max(hi - lo, 0.001), 0, 1), and sine and cosine are both multiplied by the
         # ``magnitude`` 0.1 * ln(factor) + 1.
+        # scaling = {factor} alone divides every frequency by it (positions stretched evenly).
+        self.stretch = 1.0
+        if scaling and set(scaling) == {"factor"}:
+            self.stretch, scaling = float(scaling["factor"]), None
         self.ramp = None
         if scaling and "fast" in scaling:
             self.ramp = {k: float(scaling[k]) for k in ("factor", "original", "fast", "slow")}
@@ -67,6 +71,9 @@ class RotaryEncoding(Part):
             blended = (1.0 - s) * f / c["factor"] + s * f
             f = np.where(wavelength < c["original"] / c["high"], f, np.where(wavelength > c["original"] / c["low"], f / c["factor"], blended))
             return f.astype(np.float32)
+        if self.stretch != 1.0:
+            f = np.power(np.float64(self.theta), -2.0 * np.arange(half, dtype=np.float64) / max(self.rotary_dims, 1))
+            return (f / self.stretch).astype(np.float32)
         exponent = -(np.arange(half, dtype=np.float32) * np.float32(2.0) / np.float32(self.rotary_dims))
         return np.power(np.float32(self.theta), exponent, dtype=np.float32)
 

@@ -25,6 +25,7 @@ BEFORE_THE_CHAIN = {
     "mix_w", "out_w", "in_w", "mu", "w0", "u",
     # the step's per-request metadata; norm weights over all heads, weights of a pair of mixers, the pair table
     "seq_q_start", "seq_q_len", "seq_slot", "a_bias", "q_weight", "k_weight", "wa", "wb", "pairs",
+    "blend",  # factors of the blend with the previous token's row
 }
 
 

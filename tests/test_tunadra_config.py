@@ -45,7 +45,7 @@ def test_recipe_reads_every_size_from_the_configuration():
     assert (first.feed_forward.experts, first.feed_forward.top, first.feed_forward.group_count, first.feed_forward.group_keep) == (5, 1, 5, 3)
     assert first.feed_forward.shared_size == 0 and first.feed_forward.route_scale == 0.7
     assert (second.mixer.heads, second.mixer.kv_heads, second.mixer.dim, second.mixer.vdim, second.mixer.scale) == (5, 1, 72, 40, 0.35)
-    assert second.mixer.row_dim == 128 and model.blocks[3].mixer.row_dim == 144 and second.mixer.values is None
+    assert second.mixer.row_dim == 128 and model.blocks[3].mixer.row_dim == 192 and second.mixer.values is None
     assert (second.feed_forward.group_count, second.feed_forward.limit) == (1, 0.8)
     assert model.blocks[2].feed_forward is None and model.head.softcap == 7.5 and model.embedding.scale == 0.6
     # the first layer that mixes values gives them, the later ones blend; a layer between them does neither

@@ -54,7 +54,7 @@ def test_recipe_reads_every_size_from_the_configuration():
     assert latent.cache_spec().head_dim == 9 and latent.cache_spec().planes == 1
     assert (chunked.heads, chunked.kv_heads, chunked.dim, chunked.values_from_keys, chunked.qk_bias, chunked.gate) == (5, 5, 8, True, True, "head")
     assert (chunked.chunk, chunked.softcap, chunked.position) == (0, 0.0, None)
-    assert (biased.dim, biased.vdim, biased.row_dim, biased.softcap, biased.bias_reach, biased.bias_rows) == (8, 136, 144, 2.0, 9, 6)
+    assert (biased.dim, biased.vdim, biased.row_dim, biased.softcap, biased.bias_reach, biased.bias_rows) == (8, 136, 192, 2.0, 9, 6)
     assert not biased.values_from_keys and biased.gate is None and not biased.qk_bias
     assert second_latent.position.theta == 1000.0 and second_latent.position.ramp["factor"] == 2.0
     first = model.blocks[0].feed_forward
