@@ -356,8 +356,30 @@ def zetizen_shape(width: int) -> dict:
             "layers": [biased, chunked, latent, biased][:DESIGN_LAYERS]}
 
 
-DESIGN_SHAPES = {"gunedra": gunedra_shape, "tunadra": tunadra_shape, "lerorax": lerorax_shape, "zetizen": zetizen_shape}
-CLOSEST = {"lerorax": "gunedra", "zetizen": "tunadra"}  # the existing design each is put beside by default (others: the Qwen2 shape)
+def dugalix_shape(width: int) -> dict:
+    """Layer sizes in the proportions of a real model of this design: attention heads of 128 sharing key/value heads as
+    the Qwen2 shape does, in windows of 1,024 positions, one kind with a softmax and 64 kept first tokens beside a matrix
+    memory with heads of 128 x 128, the other with sigmoid weights and a quarter of each head rotated; in the first layer
+    a dense squared-relu feed-forward, else 32 experts (plus 8 identity experts, four groups, two kept, four per token)
+    and a shared expert, sized so that a token passes through as many feed-forward weights as in the dense shape of this
+    width (ungated units have two matrices instead of three)."""
+    heads, ff = DESIGN_SIZES[width]
+    dense = {"kind": "dense", "ff": ff * 3 // 2}
+    mlp = {"kind": "moe", "expert": {"ff": ff * 3 // 16}, "shared": {"ff": ff * 3 // 4},
+           "router": {"experts": 32, "identity": 8, "top": 4, "groups": {"count": 4, "keep": 2}}}
+    kv_heads = max(1, heads // 6)
+    sizes = {"heads": heads, "kv_heads": kv_heads, "dim": 128, "vdim": 128, "scale": 128 ** -0.5}
+    pair = {"left_scale": 0.9, "right_scale": 0.7,
+            "left": dict(sizes, mask={"size": 1024, "keep_first": 64}, rot={"dims": 128, "base": 1e6, "scaling": {"factor": 8.0}}),
+            "right": {"heads": heads, "dim": 128, "vdim": 128, "gate_cap": 12.0}}
+    first = {"type": "parallel", "mlp": dense, "mixer": pair}
+    attention = {"type": "attention", "mlp": mlp, "mixer": dict(sizes, mask={"size": 1024}, rot={"dims": 32, "base": 1e6})}
+    return {"architecture": "Dugalix", "vocab": DESIGN_VOCAB, "width": width, "residual_mult": 0.5, "norm": {"eps": 1e-5},
+            "layers": [first, attention, dict(first, mlp=mlp), attention][:DESIGN_LAYERS]}
+
+
+DESIGN_SHAPES = {"dugalix": dugalix_shape, "gunedra": gunedra_shape, "tunadra": tunadra_shape, "lerorax": lerorax_shape, "zetizen": zetizen_shape}
+CLOSEST = {"lerorax": "gunedra", "zetizen": "tunadra", "dugalix": "tunadra"}  # the existing design each is put beside by default (others: the Qwen2 shape)
 # The design each is put beside: the Qwen2 shape of equal width, or (--beside) another design's shape of equal width.
 
 
@@ -532,11 +554,12 @@ def main() -> int:
                         help="instead of the headline run: prefill and decode of another design (--design) beside the Qwen2 shape of "
                         "equal width, feed-forward and head count, at a few layer sizes, with each kernel's time")
     parser.add_argument("--design-sizes", default="1536,3584", help="widths for --designs (1536, 3584 or 5120)")
-    parser.add_argument("--design", choices=["gunedra", "tunadra", "lerorax", "zetizen"], default="gunedra", help="which design --designs puts beside the Qwen2 shape")
+    parser.add_argument("--design", choices=sorted(DESIGN_SHAPES), default="gunedra", help="which design --designs puts beside the Qwen2 shape")
     parser.add_argument("--beside", choices=["qwen2", "gunedra", "tunadra"], default=None,
                         help="--designs: the shape of equal width to put the design beside (default: qwen2; for lerorax gunedra, the "
                         "closest design: blocks that norm their branches' outputs, a delta rule, short convolutions, a dense feed-forward; for "
-                        "zetizen tunadra: attention mixers over the paged cache beside a routed feed-forward with a shared expert)")
+                        "zetizen and dugalix tunadra: attention mixers over the paged cache, a routed feed-forward with a shared expert, "
+                        "and in tunadra as in dugalix a recurrent mixer with a matrix state)")
     args = parser.parse_args()
     if args.impl == "reference":
         return reference_arm(args)

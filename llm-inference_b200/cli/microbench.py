@@ -224,7 +224,7 @@ def bench_attention(args, decode: bool, mixed: bool = False) -> dict:
     for _ in range(max(1, args.layers)):
         keys = torch.randn(num_pages, kv_heads, page, dim, device="cuda").to(torch.bfloat16)
         values = torch.randn_like(keys)
-        view = CacheView(0, True, keys, values, table, num_pages, tables.shape[1], page, args.window)
+        view = CacheView(0, True, keys, values, table, num_pages, tables.shape[1], page, args.window, args.keep_first)
         if mixed:
             planes = torch.empty(kv_heads, len(positions), q_heads * dim, device="cuda", dtype=torch.bfloat16)
             talk = torch.randn(q_heads, q_heads, device="cuda")
@@ -237,7 +237,8 @@ def bench_attention(args, decode: bool, mixed: bool = False) -> dict:
             fns.append(passes)
             continue
         bias = torch.randn(q_heads, args.bias_reach + 1, device="cuda") if args.bias_reach else None
-        shape = ops.ScoreShape(args.softcap, bias, args.chunk, bias.max(dim=1).values.contiguous() if bias is not None else None)
+        shape = ops.ScoreShape(args.softcap, bias, args.chunk, bias.max(dim=1).values.contiguous() if bias is not None else None,
+                               torch.zeros(q_heads, device="cuda") if args.sigmoid else None)
         fns.append(lambda view=view, shape=shape: attention_dispatch.attend(ctx, view, q, out, q_heads, kv_heads, dim, dim**-0.5, shape=shape))
     # --rotate: back to back inside a CUDA graph, so that neither the host's launch cost nor
     # the idle gap before a lone launch enters (with one arena the cache stays in L2, as it
@@ -245,10 +246,14 @@ def bench_attention(args, decode: bool, mixed: bool = False) -> dict:
     us = time_back_to_back(fns, 16 * len(fns)) if args.rotate else time_launches(fns[0], args.iters)
     kv_bytes = sum(lens) * kv_heads * dim * 2 * 2
     flops = sum(4.0 * q_heads * dim * r * (s + (r + 1) / 2) for s, r in zip(starts, runs)) * (kv_heads if mixed else 1)
+    if args.window and not mixed:  # keys a row sees: its window, and the kept ones in front of it
+        seen = [min(p + 1, args.window) + min(args.keep_first, max(0, p + 1 - args.window)) for p in positions]
+        flops = sum(4.0 * q_heads * dim * n for n in seen)
+        kv_bytes = sum(min(n, args.window + args.keep_first) for n in lens) * kv_heads * dim * 2 * 2 if decode else kv_bytes
     if args.chunk and not mixed:
         flops = sum(4.0 * q_heads * dim * (p % args.chunk + 1) for p in positions)
     return {"kernel": ("mixed_" if mixed else "") + ("decode_attention" if decode else "prefill_attention"), "batch": len(lens), "context": args.context,
-            "tokens": len(positions), "softcap": args.softcap, "bias_reach": args.bias_reach, "chunk": args.chunk, "loader": args.loader, "splits": args.splits, "stages": args.stages,
+            "tokens": len(positions), "softcap": args.softcap, "bias_reach": args.bias_reach, "chunk": args.chunk, "window": args.window, "keep_first": args.keep_first, "sigmoid": args.sigmoid, "loader": args.loader, "splits": args.splits, "stages": args.stages,
             "layers": args.layers, "us": us, "GBps": kv_bytes / us / 1e3, "TFLOPs": flops / us / 1e6}
 
 
@@ -347,6 +352,29 @@ def bench_wkv_recurrence(args) -> dict:
     moved = 4.0 * (total * (5 * heads * dim + heads) + 2 * batch * heads * dim * dim)
     return {"kernel": "wkv_recurrence", "batch": batch, "tokens": tokens, "heads": heads, "dim": dim, "us": us,
             "us_per_token": us / tokens, "GBps": moved / us / 1e3, "TFLOPs": 5.0 * total * heads * dim * dim / us / 1e6}
+
+
+def bench_mlstm(args) -> dict:
+    """The matrix memory between its products (parts/mlstm.py: gates, recurrence, norm and gate) over ``--batch`` requests of
+    ``--tokens`` tokens each: ``--q-heads`` heads with states of ``--head-dim`` x ``--vdim``. Flops: per token and head two
+    products over the state (decay and update; read-out)."""
+    from ..parts import ops
+
+    heads, dk, dv, batch, tokens = args.q_heads, args.head_dim, args.vdim, args.batch, args.tokens
+    runs, starts = [tokens] * batch, [0] * batch
+    ctx = make_ctx([p for r in runs for p in range(r)], [i for i, r in enumerate(runs) for _ in range(r)], starts, runs)
+    ctx.seq_slot = torch.arange(batch, dtype=torch.int32, device="cuda")
+    total = batch * tokens
+    widths = [heads * dk, heads * dk, heads * dv, heads * dv, heads, heads]
+    columns = tuple(sum(widths[:i]) for i in range(6))
+    proj = torch.randn(total, sum(widths), device="cuda")
+    state = [torch.zeros(batch, heads, dk, dv, device="cuda"), torch.zeros(batch, heads, dk, device="cuda"), torch.zeros(batch, heads, device="cuda")]
+    bias, norm = torch.zeros(heads, device="cuda"), torch.ones(heads * dv, device="cuda")
+    out = torch.empty(total, heads * dv, device="cuda", dtype=torch.bfloat16)
+    us = time_launches(lambda: ops.mlstm(ctx, proj, columns, bias, bias, 10.0, state, heads, dk, dv, norm, 1e-5, out), args.iters)
+    moved = 4.0 * (total * (sum(widths) + 2 * heads * dv) + 2 * batch * heads * dk * (dv + 1)) + 2.0 * total * heads * dv
+    return {"kernel": "mlstm (gates + recurrence + output)", "batch": batch, "tokens": tokens, "heads": heads, "dim": dk, "vdim": dv, "us": us,
+            "us_per_token": us / tokens, "GBps": moved / us / 1e3, "TFLOPs": 5.0 * total * heads * dk * (dv + 1) / us / 1e6}
 
 
 def bench_delta_general_recurrence(args) -> dict:
@@ -512,7 +540,7 @@ def main(argv=None) -> int:
     parser = argparse.ArgumentParser(description=__doc__.split("\n\n")[0])
     parser.add_argument("kernel", choices=["gemm", "decode_attention", "prefill_attention", "resident", "timeline",
                                            "latent_decode_attention", "latent_prefill_attention", "delta_recurrence", "wkv_recurrence",
-                                           "moe_experts", "delta_general_recurrence", "mixed_decode_attention",
+                                           "moe_experts", "mlstm", "delta_general_recurrence", "mixed_decode_attention",
                                            "mixed_prefill_attention"])
     parser.add_argument("--experts", type=int, default=32, help="moe_experts: number of experts")
     parser.add_argument("--top", type=int, default=4, help="moe_experts: experts per token")
@@ -540,6 +568,8 @@ def main(argv=None) -> int:
     parser.add_argument("--head-dim", type=int, default=128)
     parser.add_argument("--page", type=int, default=64)
     parser.add_argument("--window", type=int, default=0)
+    parser.add_argument("--keep-first", type=int, default=0, help="attention: first keys that stay visible in front of the window")
+    parser.add_argument("--sigmoid", action="store_true", help="attention: sigmoid weights instead of a softmax")
     parser.add_argument("--plain", action="store_true")
     parser.add_argument("--softcap", type=float, default=0.0, help="attention: cap of the scores (0: none)")
     parser.add_argument("--bias-reach", type=int, default=0, help="attention: a random bias by distance up to this many positions (0: none)")
@@ -567,6 +597,8 @@ def main(argv=None) -> int:
         result = bench_wkv_recurrence(args)
     elif args.kernel == "moe_experts":
         result = bench_moe_experts(args)
+    elif args.kernel == "mlstm":
+        result = bench_mlstm(args)
     elif args.kernel == "delta_general_recurrence":
         result = bench_delta_general_recurrence(args)
     elif args.kernel.startswith("mixed_"):

@@ -74,7 +74,27 @@ def _zetizen(width, vocab, blocks, heads, kv_heads, experts, top, ff):
             "layers": [biased, chunked, latent] * blocks}
 
 
+def _dugalix(width, vocab, blocks, heads, kv_heads, experts, top, ff):
+    """``blocks`` pairs of (windowed attention beside a matrix memory, attention with sigmoid weights); a dense feed-forward in
+    the first layer, routed ones with identity experts and a shared expert after it."""
+    dense = {"kind": "dense", "ff": 4 * ff}
+    mlp = {"kind": "moe", "expert": {"ff": ff}, "shared": {"ff": 2 * ff},
+           "router": {"experts": experts, "identity": experts // 4, "top": top, "groups": {"count": 2, "keep": 1}}}
+    pair = {"type": "parallel", "mlp": mlp, "mixer": {
+        "left_scale": 0.8, "right_scale": 0.6,
+        "left": {"heads": heads, "kv_heads": kv_heads, "dim": 64, "vdim": 128, "scale": 0.125, "mask": {"size": 512, "keep_first": 4},
+                 "rot": {"dims": 64, "base": 1e6, "scaling": {"factor": 2.0}}},
+        "right": {"heads": heads // 2, "dim": 64, "vdim": 128, "gate_cap": 10.0}}}
+    attention = {"type": "attention", "mlp": mlp, "mixer": {
+        "heads": heads, "kv_heads": kv_heads, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 512}, "rot": {"dims": 32, "base": 1e5}}}
+    layers = [pair, attention] * blocks
+    layers[0] = dict(pair, mlp=dense)
+    return {"architecture": "Dugalix", "vocab": vocab, "width": width, "residual_mult": 0.5, "norm": {"eps": 1e-6}, "layers": layers}
+
+
 PRESETS = {
+    "dugalix-small": _dugalix(512, 8192, 2, 8, 2, 16, 2, 256),
+    "dugalix-1b": _dugalix(2048, 32768, 6, 16, 4, 16, 2, 512),
     "zetizen-small": _zetizen(512, 8192, 2, 8, 2, 16, 2, 256),
     "zetizen-1b": _zetizen(2048, 32768, 4, 16, 4, 16, 2, 512),
     "lerorax-small": _lerorax(512, 8192, 2, 4, 2, 1024, shared=True),
