@@ -802,10 +802,13 @@ __device__ __forceinline__ int box_offset(int row, int chunk) {
   return (chunk >> 3) * 2048 + row * 128 + (((chunk & 7) ^ (row & 7)) << 4);
 }
 
-template <int FINISH>
+// FORM_SOFTMAX, FORM_KEPT or FORM_SIGMOID, as above.
+template <int FINISH, int FORM = FORM_SOFTMAX>
 __global__ void __launch_bounds__(kFlashThreads)
 paged_decode_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_constant__ CUtensorMap v_map,
                         const FlashParams p, const int stages) {
+  constexpr bool SIGMOID = FORM == FORM_SIGMOID;
+  constexpr bool KEPT = FORM == FORM_KEPT || SIGMOID;
   constexpr int kKSteps = kTmaDim / 16;
   constexpr int kDimTiles = kTmaDim / 8;
   extern __shared__ unsigned char tma_smem_raw[];
@@ -829,6 +832,11 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
   const int lo = p.window > 0 ? max(0, first_pos - p.window + 1) : 0;
   const int hi = first_pos;
   int tile_begin = lo / kTileKeys, tile_end = hi / kTileKeys + 1;
+  // The walk counts tiles: first the kept keys' tiles that the window's do not cover, then the window's.
+  const int keep = KEPT && p.window > 0 ? p.keep_first : 0;
+  const int kept_tiles = KEPT ? min((min(keep, lo) + kTileKeys - 1) / kTileKeys, tile_begin) : 0;
+  const int window_tile = tile_begin;
+  tile_begin -= kept_tiles;
   if (p.splits > 1) {
     const int tiles = tile_end - tile_begin;
     const int per_split = max(min_tiles_per_split(p.splits), (tiles + p.splits - 1) / p.splits);
@@ -837,9 +845,13 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
   }
   const int num_tiles = max(0, tile_end - tile_begin);
 
+  auto start_of = [&](int it) {  // first key of the block's tile `it`
+    const int t = tile_begin + it;
+    return (KEPT && t < window_tile ? t - (window_tile - kept_tiles) : t) * kTileKeys;
+  };
   // Page ids of the block's tiles, checked once (a tile lies inside one page).
   auto lookup = [&](int it) -> int {
-    const int page = __ldg(table + (((tile_begin + it) * kTileKeys) >> p.page_shift));
+    const int page = __ldg(table + (start_of(it) >> p.page_shift));
     if (page < 0 || page >= p.num_pages) {
       atomicOr(p.err, ERRBIT_BAD_PAGE);
       return 0;
@@ -855,18 +867,19 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
   __syncthreads();
 
   // The warp's quarter of tile `it` holds keys key0(it) .. key0(it) + 15; the tiles in which
-  // some of them lie in [lo, hi] are consecutive: [mine_begin, mine_end).
-  const int key_off = tile_begin * kTileKeys + warp * 16;
+  // some of them lie in [lo, hi] are consecutive: [mine_begin, mine_end). (With kept keys a
+  // quarter at the front or in between that nobody sees is masked like any other hidden key.)
+  auto key0 = [&](int it) { return start_of(it) + warp * 16; };
   int mine_begin = 0, mine_end = num_tiles;
-  while (mine_begin < mine_end && key_off + mine_begin * kTileKeys + 15 < lo) ++mine_begin;
-  while (mine_end > mine_begin && key_off + (mine_end - 1) * kTileKeys > hi) --mine_end;
+  while (mine_begin < mine_end && key0(mine_begin) + 15 < lo && key0(mine_begin) >= keep) ++mine_begin;
+  while (mine_end > mine_begin && key0(mine_end - 1) > hi) --mine_end;
   const int mine = mine_end - mine_begin;
 
   unsigned char* my_ring = ring + warp * stages * kWarpStageBytes;
   auto request = [&](int j) {  // lane 0 only: the warp's j-th piece into slot j % stages
     const int it = mine_begin + j;
     const int page = it < kTmaStagedTiles ? staged_pages[it] : lookup(it);
-    const int tile_start = (tile_begin + it) * kTileKeys;
+    const int tile_start = start_of(it);
     const int arena_row = (page * p.kv_heads + kv_head) * page_size + (tile_start & p.page_mask) + warp * 16;
     const int s = j % stages;
     unsigned char* dst = my_ring + s * kWarpStageBytes;
@@ -880,7 +893,7 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
   // in front on the stream, which writes the newest key.
   int requested = 0;
   while (requested < stages && requested < mine &&
-         key_off + (mine_begin + requested) * kTileKeys + 16 <= first_pos) {
+         key0(mine_begin + requested) + 16 <= first_pos) {
     if (lane == 0) request(requested);
     ++requested;
   }
@@ -912,6 +925,8 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
   for (int i = 0; i < kDimTiles; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
   const int mi = lane >> 3;
+  const float gate0 = SIGMOID && live0 ? __ldg(p.shape.sigmoid_bias + kv_head * p.group + r0) * kLog2e : 0.f;
+  const float gate1 = SIGMOID && live1 ? __ldg(p.shape.sigmoid_bias + kv_head * p.group + r1) * kLog2e : 0.f;
 
   for (int j = 0; j < mine; ++j) {
     const int slot = j % stages;
@@ -923,7 +938,7 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
     }
     const uint32_t k_base = smem_u32(my_ring + slot * kWarpStageBytes);
     const uint32_t v_base = k_base + kWarpStageBytes / 2;
-    const int key_base = key_off + (mine_begin + j) * kTileKeys;
+    const int key_base = key0(mine_begin + j);
 
     // Scores of 16 rows x 16 keys; even and odd k-steps add into accumulators of their own, so
     // that no product waits for more than three others.
@@ -955,15 +970,24 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         float v = (s[n][e] + s_odd[n][e]) * p.scale_log2;
+        if (SIGMOID) v += e < 2 ? gate0 : gate1;
         if (needs_mask) {
           const int key = key_base + n * 8 + (lane & 3) * 2 + (e & 1);
-          if (key > hi || key < lo) v = -INFINITY;
+          if (key > hi || (key < lo && (!KEPT || key >= keep))) v = -INFINITY;
         }
         s[n][e] = v;
         if (e < 2) tile_max0 = fmaxf(tile_max0, v);
         else tile_max1 = fmaxf(tile_max1, v);
       }
     }
+    uint32_t pf[4];
+    if constexpr (SIGMOID) {
+#pragma unroll
+      for (int n = 0; n < 2; ++n) {
+        pf[n * 2 + 0] = pack_bf16(sigmoid_base2(s[n][0]), sigmoid_base2(s[n][1]));
+        pf[n * 2 + 1] = pack_bf16(sigmoid_base2(s[n][2]), sigmoid_base2(s[n][3]));
+      }
+    } else {
     tile_max0 = fmaxf(tile_max0, __shfl_xor_sync(0xffffffffu, tile_max0, 1));
     tile_max0 = fmaxf(tile_max0, __shfl_xor_sync(0xffffffffu, tile_max0, 2));
     tile_max1 = fmaxf(tile_max1, __shfl_xor_sync(0xffffffffu, tile_max1, 1));
@@ -974,7 +998,6 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
     m0 = new0;
     m1 = new1;
     float sum0 = 0.f, sum1 = 0.f;
-    uint32_t pf[4];
 #pragma unroll
     for (int n = 0; n < 2; ++n) {
       const float p00 = exp2f(s[n][0] - use0), p01 = exp2f(s[n][1] - use0);
@@ -994,6 +1017,7 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
         o[i][2] *= alpha1;
         o[i][3] *= alpha1;
       }
+    }
     }
     {
       const int vrow = (mi & 1) * 8 + (lane & 7);
@@ -1020,6 +1044,10 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
   l0 += __shfl_xor_sync(0xffffffffu, l0, 2);
   l1 += __shfl_xor_sync(0xffffffffu, l1, 1);
   l1 += __shfl_xor_sync(0xffffffffu, l1, 2);
+  if (SIGMOID) {  // nothing is normalised: the merges divide by the sum of l * 2^m over the four warps and the splits, which is 1
+    m0 = m1 = 0.f;
+    l0 = l1 = 1.f / static_cast<float>(kWarps * p.splits);
+  }
   finish_decode_block<kTmaDim, FINISH>(p, ring, o, m0, l0, m1, l1, rows_total, kv_head, q_start, split);
 }
 
@@ -1232,8 +1260,8 @@ B200_API int b200_paged_decode_attention_tma(const void* q, const void* k_arena,
                                              const int* block_table, const int* seq_q_start, const int* seq_q_len,
                                              const int* seq_kv_len, int num_seqs, int max_pages, int num_pages,
                                              int q_heads, int kv_heads, int head_dim, int page_size, int window,
-                                             float scale, int splits, int stages, float* scratch, int* err,
-                                             cudaStream_t stream) {
+                                             int keep_first, float scale, int splits, int stages,
+                                             const float* sigmoid_bias, float* scratch, int* err, cudaStream_t stream) {
   if (num_seqs == 0) return 0;
   B200_REQUIRE(b200_decode_attention_tma_supported(q_heads, kv_heads, head_dim, page_size),
                "decode attention (TMA): unsupported shape (heads %d/%d, head_dim %d, page %d)", q_heads, kv_heads,
@@ -1264,14 +1292,14 @@ B200_API int b200_paged_decode_attention_tma(const void* q, const void* k_arena,
   p.page_shift = shift;
   p.page_mask = page_size - 1;
   p.window = window;
-  p.keep_first = 0;
+  p.keep_first = keep_first;
   p.splits = splits;
   p.cluster_merge = (scratch == nullptr && splits > 1) ? 1 : 0;
   p.value_head = -1;
   p.plane_tokens = 0;
   p.scale_log2 = scale * kLog2e;
   p.scale = scale;
-  p.shape = ScoreShape{0.f, nullptr, 0, 0, nullptr};
+  p.shape = ScoreShape{0.f, nullptr, 0, 0, sigmoid_bias};
   p.cap_twice_inv = 0.f;
   p.err = err;
   p.partial_out = scratch;
@@ -1280,47 +1308,55 @@ B200_API int b200_paged_decode_attention_tma(const void* q, const void* k_arena,
   const int64_t rows = static_cast<int64_t>(num_pages) * kv_heads * page_size;
   if (decode_arena_map(&k_map, k_arena, rows) != 0) return -1;
   if (decode_arena_map(&v_map, v_arena, rows) != 0) return -1;
-  static bool configured = false;
-  if (!configured) {
-    const int most = static_cast<int>(decode_tma_smem_bytes(kTmaMaxStages));
-    if (cudaFuncSetAttribute(paged_decode_tma_kernel<FINISH_WHOLE>, cudaFuncAttributeMaxDynamicSharedMemorySize, most) != cudaSuccess ||
-        cudaFuncSetAttribute(paged_decode_tma_kernel<FINISH_PARTIAL>, cudaFuncAttributeMaxDynamicSharedMemorySize, most) != cudaSuccess ||
-        cudaFuncSetAttribute(paged_decode_tma_kernel<FINISH_CLUSTER>, cudaFuncAttributeMaxDynamicSharedMemorySize, most) != cudaSuccess)
-      return b200_fail("decode attention (TMA): cannot size shared memory");
-    configured = true;
-  }
   const dim3 grid(splits, kv_heads, num_seqs);
-  cudaError_t status;
-  if (p.cluster_merge) {
-    // The splits of a (request, kv head) form one thread-block cluster and merge on chip.
-    static bool wide_clusters = false;
-    if (splits > 8 && !wide_clusters) {
-      if (cudaFuncSetAttribute(paged_decode_tma_kernel<FINISH_CLUSTER>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) != cudaSuccess)
-        return b200_fail("decode attention (TMA): clusters of %d blocks are not allowed here", splits);
-      wide_clusters = true;
+  cudaError_t status = cudaSuccess;
+  auto launch = [&](auto form) -> int {
+    constexpr int kForm = decltype(form)::value;
+    static bool configured = false;
+    if (!configured) {
+      const int most = static_cast<int>(decode_tma_smem_bytes(kTmaMaxStages));
+      if (cudaFuncSetAttribute(paged_decode_tma_kernel<FINISH_WHOLE, kForm>, cudaFuncAttributeMaxDynamicSharedMemorySize, most) != cudaSuccess ||
+          cudaFuncSetAttribute(paged_decode_tma_kernel<FINISH_PARTIAL, kForm>, cudaFuncAttributeMaxDynamicSharedMemorySize, most) != cudaSuccess ||
+          cudaFuncSetAttribute(paged_decode_tma_kernel<FINISH_CLUSTER, kForm>, cudaFuncAttributeMaxDynamicSharedMemorySize, most) != cudaSuccess)
+        return b200_fail("decode attention (TMA): cannot size shared memory");
+      configured = true;
     }
-    cudaLaunchConfig_t config = {};
-    config.gridDim = grid;
-    config.blockDim = dim3(kFlashThreads);
-    config.dynamicSmemBytes = decode_tma_smem_bytes(stages);
-    config.stream = stream;
-    cudaLaunchAttribute attributes[2];
-    attributes[0].id = cudaLaunchAttributeClusterDimension;
-    attributes[0].val.clusterDim.x = splits;
-    attributes[0].val.clusterDim.y = 1;
-    attributes[0].val.clusterDim.z = 1;
-    attributes[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-    attributes[1].val.programmaticStreamSerializationAllowed = 1;
-    config.attrs = attributes;
-    config.numAttrs = b200_overlap_enabled() ? 2 : 1;
-    status = cudaLaunchKernelEx(&config, paged_decode_tma_kernel<FINISH_CLUSTER>, k_map, v_map, p, stages);
-  } else if (splits > 1) {
-    status = launch_kernel(paged_decode_tma_kernel<FINISH_PARTIAL>, grid, dim3(kFlashThreads),
-                           decode_tma_smem_bytes(stages), stream, k_map, v_map, p, stages);
-  } else {
-    status = launch_kernel(paged_decode_tma_kernel<FINISH_WHOLE>, grid, dim3(kFlashThreads),
-                           decode_tma_smem_bytes(stages), stream, k_map, v_map, p, stages);
-  }
+    if (p.cluster_merge) {
+      // The splits of a (request, kv head) form one thread-block cluster and merge on chip.
+      static bool wide_clusters = false;
+      if (splits > 8 && !wide_clusters) {
+        if (cudaFuncSetAttribute(paged_decode_tma_kernel<FINISH_CLUSTER, kForm>, cudaFuncAttributeNonPortableClusterSizeAllowed, 1) != cudaSuccess)
+          return b200_fail("decode attention (TMA): clusters of %d blocks are not allowed here", splits);
+        wide_clusters = true;
+      }
+      cudaLaunchConfig_t config = {};
+      config.gridDim = grid;
+      config.blockDim = dim3(kFlashThreads);
+      config.dynamicSmemBytes = decode_tma_smem_bytes(stages);
+      config.stream = stream;
+      cudaLaunchAttribute attributes[2];
+      attributes[0].id = cudaLaunchAttributeClusterDimension;
+      attributes[0].val.clusterDim.x = splits;
+      attributes[0].val.clusterDim.y = 1;
+      attributes[0].val.clusterDim.z = 1;
+      attributes[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+      attributes[1].val.programmaticStreamSerializationAllowed = 1;
+      config.attrs = attributes;
+      config.numAttrs = b200_overlap_enabled() ? 2 : 1;
+      status = cudaLaunchKernelEx(&config, paged_decode_tma_kernel<FINISH_CLUSTER, kForm>, k_map, v_map, p, stages);
+    } else if (splits > 1) {
+      status = launch_kernel(paged_decode_tma_kernel<FINISH_PARTIAL, kForm>, grid, dim3(kFlashThreads),
+                             decode_tma_smem_bytes(stages), stream, k_map, v_map, p, stages);
+    } else {
+      status = launch_kernel(paged_decode_tma_kernel<FINISH_WHOLE, kForm>, grid, dim3(kFlashThreads),
+                             decode_tma_smem_bytes(stages), stream, k_map, v_map, p, stages);
+    }
+    return 0;
+  };
+  const int refused = sigmoid_bias != nullptr              ? launch(std::integral_constant<int, FORM_SIGMOID>{})
+                      : window > 0 && keep_first > 0 ? launch(std::integral_constant<int, FORM_KEPT>{})
+                                                           : launch(std::integral_constant<int, FORM_SOFTMAX>{});
+  if (refused != 0) return refused;
   if (status != cudaSuccess) return b200_fail("decode attention (TMA): %s", cudaGetErrorString(status));
   if (splits > 1 && !p.cluster_merge) {
     status = launch_merge<kTmaDim>(p.partial_out, p.partial_ml, p.out, num_seqs * q_heads, splits, stream);

@@ -36,7 +36,7 @@ struct SkinnyStages {
   static constexpr int value = MT == 1 ? 12 : 8;
 };
 
-enum : int { EPI_BF16 = 0, EPI_F32 = 1, EPI_SWIGLU = 2 };
+enum : int { EPI_BF16 = 0, EPI_F32 = 1, EPI_SWIGLU = 2, EPI_SQUARED_RELU = 3 };
 
 __device__ __forceinline__ void mma_bf16_16816(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2,
                                                uint32_t a3, uint32_t b0, uint32_t b1) {
@@ -250,7 +250,7 @@ skinny_gemm_kernel(const __nv_bfloat16* __restrict__ W, const __nv_bfloat16* X,
       if (n >= N) continue;
       const float sum = total(r, m);
       if constexpr (EPI == EPI_F32) static_cast<float*>(Y)[static_cast<int64_t>(m) * N + n] = sum;
-      else static_cast<__nv_bfloat16*>(Y)[static_cast<int64_t>(m) * N + n] = __float2bfloat16_rn(sum);
+      else static_cast<__nv_bfloat16*>(Y)[static_cast<int64_t>(m) * N + n] = __float2bfloat16_rn(EPI == EPI_SQUARED_RELU ? fmaxf(sum, 0.f) * fmaxf(sum, 0.f) : sum);
     }
   }
 }
@@ -328,6 +328,8 @@ int launch_skinny(const __nv_bfloat16* W, const __nv_bfloat16* X, void* Y, int M
       return launch_skinny_epilogue<MT, EPI_F32>(W, X, Y, M, N, K, plan, scratch, counters, stream, ordered, fold);
     case EPI_SWIGLU:
       return launch_skinny_epilogue<MT, EPI_SWIGLU>(W, X, Y, M, N, K, plan, scratch, counters, stream, ordered, fold);
+    case EPI_SQUARED_RELU:  // not around a folded norm (the callers refuse that)
+      return launch_skinny_as<MT, EPI_SQUARED_RELU, false>(W, X, Y, M, N, K, plan, scratch, counters, stream, ordered, fold);
     default:
       return launch_skinny_epilogue<MT, EPI_BF16>(W, X, Y, M, N, K, plan, scratch, counters, stream, ordered, fold);
   }
@@ -400,7 +402,8 @@ static int skinny_gemm_run(const void* W, const void* X, void* Y, int M, int N, 
                            int64_t scratch_floats, int* counters, int num_counters, const NormFold& fold,
                            cudaStream_t stream) {
   B200_REQUIRE(b200_skinny_gemm_supported(M, N, K, epilogue), "skinny_gemm: unsupported shape %d x %d x %d", M, N, K);
-  B200_REQUIRE(epilogue >= EPI_BF16 && epilogue <= EPI_SWIGLU, "skinny_gemm: unknown epilogue %d", epilogue);
+  B200_REQUIRE(epilogue >= EPI_BF16 && epilogue <= EPI_SQUARED_RELU, "skinny_gemm: unknown epilogue %d", epilogue);
+  B200_REQUIRE(epilogue != EPI_SQUARED_RELU || (fold.ss_in == nullptr && fold.x == nullptr), "skinny_gemm: the squared relu has no folded form");
   B200_REQUIRE(reinterpret_cast<uintptr_t>(W) % 16 == 0 && reinterpret_cast<uintptr_t>(X) % 16 == 0,
                "skinny_gemm: operands must be 16-byte aligned");
   const SkinnyPlan plan = plan_skinny(N, K);
@@ -471,7 +474,7 @@ B200_API int b200_skinny_gemm_static(const void* W, const void* X, void* Y, int 
                                      cudaStream_t stream) {
   B200_REQUIRE(b200_skinny_gemm_supported(M, N, K, epilogue),
                "skinny_gemm_static: unsupported shape %d x %d x %d (at most 16 rows, K a multiple of 8)", M, N, K);
-  B200_REQUIRE(epilogue >= EPI_BF16 && epilogue <= EPI_SWIGLU, "skinny_gemm_static: unknown epilogue %d", epilogue);
+  B200_REQUIRE(epilogue >= EPI_BF16 && epilogue <= EPI_SQUARED_RELU, "skinny_gemm_static: unknown epilogue %d", epilogue);
   B200_REQUIRE(W != nullptr && X != nullptr && Y != nullptr, "skinny_gemm_static: null operand");
   B200_REQUIRE(reinterpret_cast<uintptr_t>(W) % 16 == 0 && reinterpret_cast<uintptr_t>(X) % 16 == 0,
                "skinny_gemm_static: operands must be 16-byte aligned");

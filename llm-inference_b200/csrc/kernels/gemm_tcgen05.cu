@@ -55,7 +55,7 @@ constexpr int kThreadsT = 192;   // warp 0: TMA, warp 1: MMA, warps 2-5: epilogu
 constexpr long long kWaitCycles = 4000000000LL;  // about two seconds
 constexpr int ERRBIT_TIMEOUT = 8;
 
-enum : int { EPI_BF16 = 0, EPI_F32 = 1, EPI_SWIGLU = 2 };
+enum : int { EPI_BF16 = 0, EPI_F32 = 1, EPI_SWIGLU = 2, EPI_SQUARED_RELU = 3 };
 
 __device__ __forceinline__ uint32_t smem_addr(const void* p) {
   return static_cast<uint32_t>(__cvta_generic_to_shared(p));
@@ -161,7 +161,7 @@ enum : int { MODE_SINGLE = 0, MODE_PUSH = 1, MODE_PULL = 2 };
 template <int EPI>
 __device__ __forceinline__ void write_output(const StreamParams& p, int m, int n, float v) {
   if constexpr (EPI == EPI_F32) static_cast<float*>(p.y)[static_cast<int64_t>(m) * p.N + n] = v;
-  else static_cast<__nv_bfloat16*>(p.y)[static_cast<int64_t>(m) * p.N + n] = __float2bfloat16_rn(v);
+  else static_cast<__nv_bfloat16*>(p.y)[static_cast<int64_t>(m) * p.N + n] = __float2bfloat16_rn(EPI == EPI_SQUARED_RELU ? fmaxf(v, 0.f) * fmaxf(v, 0.f) : v);
 }
 
 // A cluster member's slice of the rows, added up over the members' partial tiles
@@ -631,6 +631,10 @@ StreamKernel pick_kernel(int epilogue, int mode, bool folded, bool traced) {
   switch (epilogue) {
     case EPI_F32: return pick_mode<EPI_F32>(mode, folded, traced);
     case EPI_SWIGLU: return pick_mode<EPI_SWIGLU>(mode, folded, traced);
+    case EPI_SQUARED_RELU:  // plain form only: not around a folded norm (refused), not traced
+      return mode == MODE_SINGLE ? stream_gemm_kernel<EPI_SQUARED_RELU, MODE_SINGLE, false, false>
+             : mode == MODE_PUSH ? stream_gemm_kernel<EPI_SQUARED_RELU, MODE_PUSH, false, false>
+                                 : stream_gemm_kernel<EPI_SQUARED_RELU, MODE_PULL, false, false>;
     default: return pick_mode<EPI_BF16>(mode, folded, traced);
   }
 }
@@ -850,7 +854,8 @@ B200_API int b200_stream_gemm_fold(const void* W, const void* X, void* Y, int M,
 static int stream_gemm_run(const void* W, const void* X, void* Y, int M, int N, int K, int epilogue, int* err,
                            const NormFold& fold, cudaStream_t stream) {
   B200_REQUIRE(b200_stream_gemm_supported(M, N, K, epilogue), "stream_gemm: unsupported shape %d x %d x %d", M, N, K);
-  B200_REQUIRE(epilogue >= EPI_BF16 && epilogue <= EPI_SWIGLU, "stream_gemm: unknown epilogue %d", epilogue);
+  B200_REQUIRE(epilogue >= EPI_BF16 && epilogue <= EPI_SQUARED_RELU, "stream_gemm: unknown epilogue %d", epilogue);
+  B200_REQUIRE(epilogue != EPI_SQUARED_RELU || (fold.ss_in == nullptr && fold.x == nullptr), "stream_gemm: the squared relu has no folded form");
   B200_REQUIRE(reinterpret_cast<uintptr_t>(W) % 16 == 0 && reinterpret_cast<uintptr_t>(X) % 16 == 0,
                "stream_gemm: operands must be 16-byte aligned");
   StreamParams p;

@@ -26,6 +26,7 @@
 #include <type_traits>
 
 #include "common.cuh"
+#include "packs.cuh"
 
 namespace {
 
@@ -508,23 +509,26 @@ moe_down_mma_kernel(const __nv_bfloat16* act, const __nv_bfloat16* __restrict__ 
 // out[t] = sum_j weights[t][j] * expert_out[t * top + j] (+ shared[t]), in the order of j. IDENTITY: a choice whose id is at or
 // past `experts` is an identity expert, whose output is h[t]. With `gate` (rows `gate_ld` apart) the shared expert's output is
 // multiplied by sigmoid(gate[t]).
-template <typename T, bool IDENTITY>
+template <typename T, bool IDENTITY, int W>
 __global__ void moe_combine_kernel(const float* expert_out, const float* weights, const T* shared, const int* ids, int experts, const T* h,
                                    const float* gate, int gate_ld, int top, int width, T* out) {
   wait_for_predecessor();
   let_successor_start();
+  using P = Pack<W>;
+  using V = typename P::type;
   const int t = blockIdx.x;
   const float share = gate ? sigmoid_f(gate[static_cast<int64_t>(t) * gate_ld]) : 1.f;
-  for (int d = threadIdx.x; d < width; d += blockDim.x) {
-    float acc = 0.f;
-    const float own = IDENTITY ? to_f32<T>(h[static_cast<int64_t>(t) * width + d]) : 0.f;
+  const int64_t row = static_cast<int64_t>(t) * width, first = static_cast<int64_t>(t) * top;
+  for (int d = threadIdx.x * W; d < width; d += blockDim.x * W) {
+    V acc = {};
+    V own = {};
+    if (IDENTITY) own = P::load(h + row + d);
     for (int j = 0; j < top; ++j) {
-      const int64_t slot = static_cast<int64_t>(t) * top + j;
-      const float y = IDENTITY && ids[slot] >= experts ? own : expert_out[slot * width + d];
-      acc = fmaf(weights[slot], y, acc);
+      const V y = IDENTITY && ids[first + j] >= experts ? own : P::load(expert_out + (first + j) * width + d);
+      acc = fma_each(y, weights[first + j], acc);
     }
-    if (shared) acc = fmaf(share, to_f32<T>(shared[static_cast<int64_t>(t) * width + d]), acc);
-    out[static_cast<int64_t>(t) * width + d] = from_f32<T>(acc);
+    if (shared) acc = fma_each(P::load(shared + row + d), share, acc);
+    P::store(out + row + d, acc);
   }
 }
 
@@ -698,18 +702,25 @@ B200_API int b200_moe_combine(const float* expert_out, const float* weights, con
                               const float* gate, int gate_ld, int tokens, int top, int width, void* out, int dtype, cudaStream_t stream) {
   if (tokens == 0) return 0;
   B200_REQUIRE(tokens > 0 && top > 0 && width > 0 && (ids == nullptr || h != nullptr), "moe_combine: bad sizes");
-  const int threads = width >= 1024 ? 256 : 128;
+  const bool wide = packs_of_four(width, expert_out, shared, h, out);
+  const int packs = wide ? width / 4 : width;
+  const int threads = packs >= 512 ? 256 : 128;
   auto launch = [&](auto kernel, auto* typed) {
     using T = std::remove_pointer_t<decltype(typed)>;
     launch_kernel(kernel, dim3(tokens), dim3(threads), 0, stream, expert_out, weights, static_cast<const T*>(shared), ids, experts,
                   static_cast<const T*>(h), gate, gate_ld, top, width, typed);
   };
+  auto pick = [&](auto* typed) {
+    using T = std::remove_pointer_t<decltype(typed)>;
+    if (ids && wide) launch(moe_combine_kernel<T, true, 4>, typed);
+    else if (ids) launch(moe_combine_kernel<T, true, 1>, typed);
+    else if (wide) launch(moe_combine_kernel<T, false, 4>, typed);
+    else launch(moe_combine_kernel<T, false, 1>, typed);
+  };
   if (dtype == DTYPE_F32) {
-    if (ids) launch(moe_combine_kernel<float, true>, static_cast<float*>(out));
-    else launch(moe_combine_kernel<float, false>, static_cast<float*>(out));
+    pick(static_cast<float*>(out));
   } else if (dtype == DTYPE_BF16) {
-    if (ids) launch(moe_combine_kernel<__nv_bfloat16, true>, static_cast<__nv_bfloat16*>(out));
-    else launch(moe_combine_kernel<__nv_bfloat16, false>, static_cast<__nv_bfloat16*>(out));
+    pick(static_cast<__nv_bfloat16*>(out));
   } else {
     return b200_fail("moe_combine: unknown dtype %d", dtype);
   }

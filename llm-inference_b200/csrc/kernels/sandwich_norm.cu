@@ -13,6 +13,7 @@
 // 1 / rms(x) per row and copies the slots of the step's requests aside, and `shift_norm` forms h_t and h_(t-1) from the
 // stream's rows, blends them and moves the slots on. Both ways round the blend once, at the end.
 #include "common.cuh"
+#include "packs.cuh"
 
 namespace {
 
@@ -38,68 +39,6 @@ struct SandwichParams {
   const int* seq_slot;
   float* rstd_out;         // [tokens], SHIFT_DEFER
   float* previous;         // [requests][hidden], SHIFT_DEFER: the slots as they were before the step
-};
-
-template <typename T>
-__device__ __forceinline__ float4 load4(const T* p);
-template <>
-__device__ __forceinline__ float4 load4<float>(const float* p) { return *reinterpret_cast<const float4*>(p); }
-template <>
-__device__ __forceinline__ float4 load4<__nv_bfloat16>(const __nv_bfloat16* p) {
-  const uint2 raw = *reinterpret_cast<const uint2*>(p);
-  const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
-  const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
-  return make_float4(lo.x, lo.y, hi.x, hi.y);
-}
-template <typename T>
-__device__ __forceinline__ void store4(T* p, float4 v);
-template <>
-__device__ __forceinline__ void store4<float>(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
-template <>
-__device__ __forceinline__ void store4<__nv_bfloat16>(__nv_bfloat16* p, float4 v) {
-  __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
-  uint2 raw;
-  raw.x = *reinterpret_cast<uint32_t*>(&lo);
-  raw.y = *reinterpret_cast<uint32_t*>(&hi);
-  *reinterpret_cast<uint2*>(p) = raw;
-}
-// One number as a "vector" of one, so that rows of any length share the code below.
-template <typename T>
-__device__ __forceinline__ float load1(const T* p) { return to_f32<T>(*p); }
-
-__device__ __forceinline__ float fma_each(float a, float b, float c) { return fmaf(a, b, c); }
-__device__ __forceinline__ float4 fma_each(float4 a, float4 b, float4 c) {
-  return make_float4(fmaf(a.x, b.x, c.x), fmaf(a.y, b.y, c.y), fmaf(a.z, b.z, c.z), fmaf(a.w, b.w, c.w));
-}
-__device__ __forceinline__ float scale_each(float a, float s) { return a * s; }
-__device__ __forceinline__ float4 scale_each(float4 a, float s) { return make_float4(a.x * s, a.y * s, a.z * s, a.w * s); }
-__device__ __forceinline__ float mul_each(float a, float b) { return a * b; }
-__device__ __forceinline__ float4 mul_each(float4 a, float4 b) { return make_float4(a.x * b.x, a.y * b.y, a.z * b.z, a.w * b.w); }
-__device__ __forceinline__ float add_each(float a, float b) { return a + b; }
-__device__ __forceinline__ float4 add_each(float4 a, float4 b) { return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w); }
-__device__ __forceinline__ float sub_each(float a, float b) { return a - b; }
-__device__ __forceinline__ float4 sub_each(float4 a, float4 b) { return make_float4(a.x - b.x, a.y - b.y, a.z - b.z, a.w - b.w); }
-__device__ __forceinline__ float square_sum(float a, float acc) { return fmaf(a, a, acc); }
-__device__ __forceinline__ float square_sum(float4 a, float acc) { return fmaf(a.x, a.x, fmaf(a.y, a.y, fmaf(a.z, a.z, fmaf(a.w, a.w, acc)))); }
-
-// W numbers per access: 4 (rows whose length is a multiple of four, aligned) or 1.
-template <int W>
-struct Pack;
-template <>
-struct Pack<4> {
-  using type = float4;
-  template <typename T>
-  static __device__ __forceinline__ float4 load(const T* p) { return load4<T>(p); }
-  template <typename T>
-  static __device__ __forceinline__ void store(T* p, float4 v) { store4<T>(p, v); }
-};
-template <>
-struct Pack<1> {
-  using type = float;
-  template <typename T>
-  static __device__ __forceinline__ float load(const T* p) { return load1<T>(p); }
-  template <typename T>
-  static __device__ __forceinline__ void store(T* p, float v) { *p = from_f32<T>(v); }
 };
 
 // PER packs of W numbers a thread, in registers; PER = 0: any row length, the row in shared memory.
@@ -211,8 +150,6 @@ __global__ void shift_norm_kernel(const float* x, const float* rstd, const float
   }
 }
 
-bool aligned16(const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; }
-
 template <typename T, int W, int PER, int SHIFT>
 void launch_sandwich(const SandwichParams& p, int count, int threads, cudaStream_t stream) {
   const size_t smem = PER == 0 ? sizeof(float) * p.hidden : 0;
@@ -223,12 +160,14 @@ void launch_sandwich(const SandwichParams& p, int count, int threads, cudaStream
 
 template <typename T, int SHIFT>
 void sandwich_by_width(const SandwichParams& p, int count, bool wide, cudaStream_t stream) {
-  if (wide && p.hidden <= 4096) {  // up to two packs of four a thread, whole warps
-    const int threads = p.hidden <= 1024 ? (p.hidden / 4 + 31) / 32 * 32 : (p.hidden / 8 + 31) / 32 * 32;
-    if (p.hidden <= 1024) launch_sandwich<T, 4, 1, SHIFT>(p, count, threads, stream);
-    else launch_sandwich<T, 4, 2, SHIFT>(p, count, threads, stream);
+  // Whole warps, at most `per` packs of four a thread.
+  auto threads_for = [&](int per) { return ((p.hidden / 4 + per - 1) / per + 31) / 32 * 32; };
+  if (wide && p.hidden <= 1024) {
+    launch_sandwich<T, 4, 1, SHIFT>(p, count, threads_for(1), stream);
+  } else if (wide && p.hidden <= 4096) {
+    launch_sandwich<T, 4, 2, SHIFT>(p, count, threads_for(2), stream);
   } else if (wide && p.hidden <= 8192) {
-    launch_sandwich<T, 4, 4, SHIFT>(p, count, (p.hidden / 16 + 31) / 32 * 32, stream);
+    launch_sandwich<T, 4, 4, SHIFT>(p, count, threads_for(4), stream);
   } else if (wide) {
     launch_sandwich<T, 4, 0, SHIFT>(p, count, 512, stream);
   } else {
@@ -263,11 +202,7 @@ B200_API int b200_sandwich_norm(float* x, const void* a, const void* b, float a_
   B200_REQUIRE(mode == SHIFT_DEFER || out != nullptr, "sandwich_norm: no output");
   SandwichParams p{x, a, b, a_scale, b_scale, constant, branch_weight, mult, branch_eps, weight, eps, rows, hidden, out,
                    shift, slots, token_seq, seq_q_start, seq_slot, rstd_out, previous};
-  bool wide = hidden % 4 == 0;
-  for (const void* q : {static_cast<const void*>(x), a, b, static_cast<const void*>(constant), static_cast<const void*>(branch_weight),
-                        static_cast<const void*>(weight), static_cast<const void*>(out), static_cast<const void*>(shift),
-                        static_cast<const void*>(slots), static_cast<const void*>(previous)})
-    wide = wide && aligned16(q);
+  const bool wide = packs_of_four(hidden, x, a, b, constant, branch_weight, weight, out, shift, slots, previous);
   if (dtype == DTYPE_F32) sandwich_by_mode<float>(p, count, wide, mode, stream);
   else if (dtype == DTYPE_BF16) sandwich_by_mode<__nv_bfloat16>(p, count, wide, mode, stream);
   else return b200_fail("sandwich_norm: unknown dtype %d", dtype);
@@ -279,10 +214,7 @@ B200_API int b200_shift_norm(const float* x, const float* rstd, const float* wei
                              void* out, int dtype, cudaStream_t stream) {
   if (tokens == 0) return 0;
   B200_REQUIRE(tokens > 0 && hidden > 0, "shift_norm: bad sizes");
-  bool wide = hidden % 4 == 0;
-  for (const void* q : {static_cast<const void*>(x), static_cast<const void*>(weight), static_cast<const void*>(shift),
-                        static_cast<const void*>(previous), static_cast<const void*>(slots), static_cast<const void*>(out)})
-    wide = wide && aligned16(q);
+  const bool wide = packs_of_four(hidden, x, weight, shift, previous, slots, out);
   auto launch = [&](auto kernel, auto* typed) {
     const int packs = wide ? hidden / 4 : hidden;
     const int threads = packs >= 256 ? 256 : (packs + 31) / 32 * 32;

@@ -10,6 +10,9 @@
 // multiplied by `magnitude`; the rest of the head passes unchanged. Queries go to a dense buffer and keys and values
 // into the token's page, all in rows of `row_dim` numbers padded with zeros (the arena has one row width for keys
 // and values). The token that starts a page clears the rows its step does not fill.
+//
+// Without norms nothing binds a token's heads together: `qk_rope_write_pairs` (bfloat16, even sizes) works out the token's
+// sines and cosines once, for all its heads, and moves two neighbouring numbers an access straight from the projection.
 #include "common.cuh"
 #include "page_tail.cuh"
 
@@ -107,6 +110,89 @@ __global__ void qk_norm_rope_write_kernel(const T* proj, int ld, const float* __
   }
 }
 
+__device__ __forceinline__ float2 pair_at(const __nv_bfloat16* row, const float* bias, int i) {
+  float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(row + i));
+  if (bias) {
+    v.x += bias[i];
+    v.y += bias[i + 1];
+  }
+  return v;
+}
+__device__ __forceinline__ void put_pair(__nv_bfloat16* dst, float2 v) { *reinterpret_cast<__nv_bfloat162*>(dst) = __floats2bfloat162_rn(v.x, v.y); }
+
+// Every size even (dim, vdim, row_dim, ld, rot_dims / 2).
+__global__ void qk_rope_write_pairs_kernel(const __nv_bfloat16* proj, int ld, const float* __restrict__ bias, const float* __restrict__ inv_freq,
+                                           int rot_dims, float magnitude, int values_from_keys, const int* __restrict__ positions,
+                                           const int* __restrict__ token_seq, const int* __restrict__ seq_kv_len,
+                                           const int* __restrict__ block_table, int max_pages, int num_pages, __nv_bfloat16* k_arena,
+                                           __nv_bfloat16* v_arena, __nv_bfloat16* q_out, int q_heads, int kv_heads, int dim, int vdim, int row_dim,
+                                           int page_size, int write_kv, int* err) {
+  extern __shared__ float2 turns[];  // [rot_dims / 2]: cosine and sine
+  let_successor_start();
+  const int t = blockIdx.x, tid = threadIdx.x;
+  const int pos = positions[t], half = rot_dims / 2;
+  for (int i = tid; i < half; i += blockDim.x) {
+    float s, c;
+    sincosf(static_cast<float>(pos) * inv_freq[i], &s, &c);
+    turns[i] = make_float2(c * magnitude, s * magnitude);
+  }
+  int page = -1, clear_from = 0;
+  if (write_kv) {
+    const int logical = pos / page_size;
+    if (pos < 0 || logical >= max_pages) {
+      if (tid == 0) atomicOr(err, ERRBIT_BAD_POSITION);
+    } else {
+      page = block_table[static_cast<int64_t>(token_seq[t]) * max_pages + logical];
+      if (page < 0 || page >= num_pages) {
+        if (tid == 0) atomicOr(err, ERRBIT_BAD_PAGE);
+        page = -1;
+      } else if (pos % page_size == 0 && seq_kv_len != nullptr) {
+        clear_from = max(1, seq_kv_len[token_seq[t]] - pos);
+      }
+    }
+  }
+  __syncthreads();
+  wait_for_predecessor();
+  const __nv_bfloat16* row = proj + static_cast<int64_t>(t) * ld;
+  const int q_width = q_heads * dim, k_width = kv_heads * dim;
+  const int64_t head_stride = static_cast<int64_t>(page_size) * row_dim;
+  const int64_t in_page = static_cast<int64_t>(pos % page_size) * row_dim;
+  __nv_bfloat16* k_tile = page >= 0 ? k_arena + kv_row_offset(page, 0, 0, kv_heads, page_size, row_dim) : nullptr;
+  __nv_bfloat16* v_tile = page >= 0 ? v_arena + kv_row_offset(page, 0, 0, kv_heads, page_size, row_dim) : nullptr;
+  if (clear_from > 0 && page >= 0) {
+    for (int h = 0; h < kv_heads; ++h) {
+      clear_page_tail(k_tile + h * head_stride, clear_from, page_size, row_dim);  // the token sits in row 0 of the page
+      clear_page_tail(v_tile + h * head_stride, clear_from, page_size, row_dim);
+    }
+  }
+  if (page >= 0) {
+    const int source = values_from_keys ? q_width : q_width + k_width, pairs = row_dim / 2;
+    for (int idx = tid; idx < kv_heads * pairs; idx += blockDim.x) {
+      const int h = idx / pairs, i = (idx - h * pairs) * 2;
+      const float2 v = i < vdim ? pair_at(row, bias, source + h * vdim + i) : make_float2(0.f, 0.f);
+      put_pair(v_tile + h * head_stride + in_page + i, v);
+    }
+  }
+  // Per head: half / 2 items of two rotated pairs, then two numbers an item of what is not rotated and of the padding.
+  const int turned = half / 2, items = turned + (row_dim - rot_dims) / 2;
+  for (int idx = tid; idx < (q_heads + kv_heads) * items; idx += blockDim.x) {
+    const int head = idx / items, i = idx - head * items;
+    const bool is_q = head < q_heads;
+    if (!is_q && page < 0) continue;
+    const int at = head * dim;  // k heads follow the q heads in the row
+    __nv_bfloat16* dst = is_q ? q_out + (static_cast<int64_t>(t) * q_heads + head) * row_dim : k_tile + (head - q_heads) * head_stride + in_page;
+    if (i < turned) {
+      const float2 u = pair_at(row, bias, at + 2 * i), v = pair_at(row, bias, at + 2 * i + half);
+      const float2 a = turns[2 * i], b = turns[2 * i + 1];
+      put_pair(dst + 2 * i, make_float2(u.x * a.x - v.x * a.y, u.y * b.x - v.y * b.y));
+      put_pair(dst + 2 * i + half, make_float2(v.x * a.x + u.x * a.y, v.y * b.x + u.y * b.y));
+    } else {
+      const int d = rot_dims + (i - turned) * 2;
+      put_pair(dst + d, d < dim ? pair_at(row, bias, at + d) : make_float2(0.f, 0.f));
+    }
+  }
+}
+
 }  // namespace
 
 B200_API int b200_qk_norm_rope_write(const void* proj, int ld, const float* bias, const float* q_weight, const float* k_weight, float eps,
@@ -122,6 +208,15 @@ B200_API int b200_qk_norm_rope_write(const void* proj, int ld, const float* bias
   B200_REQUIRE(!values_from_keys || vdim == dim, "qk_norm_rope_write: values that are the keys have the keys' size");
   B200_REQUIRE(ld >= (q_heads + kv_heads) * dim + (values_from_keys ? 0 : kv_heads * vdim),
                "qk_norm_rope_write: rows of %d numbers do not hold the projections", ld);
+  if (dtype == DTYPE_BF16 && q_weight == nullptr && k_weight == nullptr && (dim | vdim | row_dim | ld | (rot_dims / 2)) % 2 == 0) {
+    const int pairs = (q_heads + 2 * kv_heads) * row_dim / 2;
+    const int width = pairs >= 1024 ? 256 : 128;
+    launch_kernel(qk_rope_write_pairs_kernel, dim3(tokens), dim3(width), sizeof(float2) * (rot_dims / 2), stream,
+                  static_cast<const __nv_bfloat16*>(proj), ld, bias, inv_freq, rot_dims, magnitude, values_from_keys, positions, token_seq,
+                  seq_kv_len, block_table, max_pages, num_pages, static_cast<__nv_bfloat16*>(k_arena), static_cast<__nv_bfloat16*>(v_arena),
+                  static_cast<__nv_bfloat16*>(q_out), q_heads, kv_heads, dim, vdim, row_dim, page_size, write_kv, err);
+    return b200_check_launch("qk_rope_write_pairs");
+  }
   const size_t smem = sizeof(float) * (q_heads + kv_heads) * dim;
   B200_REQUIRE(smem <= 160 * 1024, "qk_norm_rope_write: %d numbers of q and k do not fit one block", (q_heads + kv_heads) * dim);
   const int work = (q_heads + kv_heads) * dim;

@@ -59,7 +59,7 @@ _SIGNATURES: dict[str, list] = {
     "b200_gemm_f32": [c_void_p] * 4 + [c_int] * 6 + [c_void_p],
     "b200_paged_flash_attention": [c_void_p] * 8 + [c_int] * 12 + [c_float, c_int, c_int, c_int, c_float, c_void_p, c_int, c_int, c_void_p,
                                    c_void_p, c_void_p, c_void_p],
-    "b200_paged_decode_attention_tma": [c_void_p] * 8 + [c_int] * 8 + [c_float, c_int, c_int, c_void_p, c_void_p, c_void_p],
+    "b200_paged_decode_attention_tma": [c_void_p] * 8 + [c_int] * 9 + [c_float, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p],
     "b200_flash_prefill_tcgen05": [c_void_p] * 8 + [c_int] * 12 + [c_float, c_int, c_float, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p,
                                    c_void_p],
     "b200_skinny_gemm": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int64, c_void_p, c_int, c_void_p],

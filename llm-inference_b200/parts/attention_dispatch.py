@@ -33,8 +33,8 @@ def attend(
     """``shape``: a soft cap, a bias by distance and a chunk of visible keys (``ops.ScoreShape``); the plain kernel, the
     mma.sync kernels and the tcgen05 prefill kernel take it. So shaped prompt portions run on tcgen05 where its sizes hold
     (heads of 128) and the mma.sync prefill form otherwise, and decoded tokens with any shaping the cp.async split-key kernel.
-    The same holds for sigmoid weights (``shape.sigmoid_bias``) and for first keys kept in front of a window
-    (``cache.keep_first``), which those kernels take as forms of their own.
+    Sigmoid weights (``shape.sigmoid_bias``) and first keys kept in front of a window (``cache.keep_first``) are forms of
+    every kernel, the TMA decode kernel's among them.
 
     ``value_head`` >= 0: every query head's weights are applied to the values of that one kv head
     instead of its own (a mixer that mixes weights over heads asks for one such pass per kv head); the
@@ -59,7 +59,7 @@ def attend(
         reach = ctx.max_kv_len if not cache.window else min(ctx.max_kv_len, cache.window + 64 + cache.keep_first)
         if shape.chunk:
             reach = min(reach, shape.chunk)  # a decoded token sees its own chunk at most
-        tma = value_head < 0 and not shape and not cache.keep_first and ops.decode_uses_tma(ctx, decode_seqs, q_heads, kv_heads, head_dim, cache.page_size)
+        tma = value_head < 0 and not shape.changes_scores() and ops.decode_uses_tma(ctx, decode_seqs, q_heads, kv_heads, head_dim, cache.page_size)
         splits = int(ctx.options.get("decode_splits", 0)) or ops.decode_splits(decode_seqs, kv_heads, reach, tma, ops.sm_count(ctx))
         ops.paged_flash_attention(
             ctx, cache, q, out, q_heads, kv_heads, head_dim, scale,

@@ -362,13 +362,16 @@ class ScoreShape:
     sigmoid_bias: torch.Tensor | None = None  # float32 [q_heads]: a visible key weighs sigmoid(score + bias), nothing is normalised
 
     def __bool__(self) -> bool:
-        return bool(self.softcap > 0.0 or self.bias is not None or self.chunk > 0 or self.sigmoid_bias is not None)
+        return self.changes_scores() or self.sigmoid_bias is not None
+
+    def changes_scores(self) -> bool:
+        """Whether a score is more than the scaled product (the TMA decode kernel takes none of that)."""
+        return bool(self.softcap > 0.0 or self.bias is not None or self.chunk > 0)
 
     def tensor_cores_take(self, cache: CacheView) -> bool:
         """The tensor-core kernels have one form per kind of score: a cap, bias or chunk does not go together with sigmoid
         weights or with first keys kept in front of a window (the plain kernel takes every combination)."""
-        changed = self.softcap > 0.0 or self.bias is not None or self.chunk > 0
-        return not (changed and (self.sigmoid_bias is not None or (cache.window and cache.keep_first)))
+        return not (self.changes_scores() and (self.sigmoid_bias is not None or (cache.window and cache.keep_first)))
 
     def arguments(self, q_heads: int) -> list:
         if self.bias is not None:
@@ -521,7 +524,7 @@ def paged_flash_attention(
     # slow to place. The TMA kernel always goes through scratch unless told otherwise: at
     # batch 1 both forms take 1.10 ms per step (the cp.async kernel 1.15), at batch 2 scratch
     # 1.10 and the cluster 1.12, from batch 4 on the cluster loses.
-    use_tma = decode and value_head == -1 and not shape and not cache.keep_first and decode_uses_tma(ctx, num_seqs, q_heads, kv_heads, head_dim, cache.page_size)
+    use_tma = decode and value_head == -1 and not shape.changes_scores() and decode_uses_tma(ctx, num_seqs, q_heads, kv_heads, head_dim, cache.page_size)
     merge = ctx.options.get("attention_merge", "auto")
     if merge == "auto":
         merge = "cluster" if num_seqs * kv_heads * planes <= 4 and not use_tma else "scratch"
@@ -534,8 +537,8 @@ def paged_flash_attention(
             "b200_paged_decode_attention_tma", ptr(q), ptr(cache.keys), ptr(cache.values), ptr(out), ptr(cache.block_table),
             ptr(ctx.seq_q_start), ptr(ctx.seq_q_len), ptr(ctx.seq_kv_len), c_int(num_seqs), c_int(cache.max_pages),
             c_int(cache.num_pages), c_int(q_heads), c_int(kv_heads), c_int(head_dim), c_int(cache.page_size),
-            c_int(cache.window), c_float(scale), c_int(splits), c_int(int(ctx.options.get("decode_stages", DECODE_STAGES))),
-            ptr(scratch), ptr(ctx.err), ctx.stream,
+            c_int(cache.window), c_int(cache.keep_first), c_float(scale), c_int(splits), c_int(int(ctx.options.get("decode_stages", DECODE_STAGES))),
+            ptr(shape.sigmoid_bias), ptr(scratch), ptr(ctx.err), ctx.stream,
         )
         if scratch is not None:
             ctx.lib.calls += 1  # the merge kernel is a launch of its own
@@ -1508,7 +1511,15 @@ def mlstm(ctx: StepContext, proj: torch.Tensor, columns: tuple[int, int, int, in
 
 
 def linear_squared_relu(ctx: StepContext, x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
-    """``out = max(x @ weight.T, 0)^2``."""
+    """``out = max(x @ weight.T, 0)^2``: the activation is an epilogue of this engine's own products of short steps, a pass
+    of its own behind the library's."""
+    m, k = x.shape
+    if x.dtype == torch.bfloat16 and m and x.is_contiguous():
+        kernel = _small_gemm_kernel(ctx, m, weight.shape[0], k, 3)
+        if kernel is not None:
+            _need(weight.shape[1] == k and tuple(out.shape) == (m, weight.shape[0]) and out.is_contiguous(), "linear_squared_relu: bad operands")
+            _small_gemm(ctx, kernel, x, weight, out, 3)
+            return out
     return squared_relu(ctx, linear(ctx, x, weight, out))
 
 
