@@ -152,9 +152,9 @@ def bench_gemm(args) -> dict:
         out = torch.empty(m, n // 2 if args.swiglu else n, device="cuda", dtype=torch.float32 if args.f32_out else torch.bfloat16)
         if args.swiglu and args.gemm == "library":
             mid = torch.empty(m, n, device="cuda", dtype=torch.bfloat16)
-            fns = [lambda wi=wi: (ops.linear(ctx, x, wi, mid), ops.silu_mul(ctx, mid, out)) for wi in weights]
+            fns = [lambda wi=wi: (ops.linear(ctx, x, wi, mid), ops.gated_mul(ctx, mid, out)) for wi in weights]
         elif args.swiglu:
-            fns = [lambda wi=wi: ops.linear_swiglu(ctx, x, wi, out) for wi in weights]
+            fns = [lambda wi=wi: ops.linear_gated(ctx, x, wi, out) for wi in weights]
         else:
             fns = [lambda wi=wi: ops.linear(ctx, x, wi, out) for wi in weights]
         if args.trace:
@@ -173,9 +173,9 @@ def bench_gemm(args) -> dict:
 
             def fn():
                 ops.linear(ctx, x, w, mid)
-                ops.silu_mul(ctx, mid, out)
+                ops.gated_mul(ctx, mid, out)
         else:
-            fn = lambda: ops.linear_swiglu(ctx, x, w, out)
+            fn = lambda: ops.linear_gated(ctx, x, w, out)
     else:
         out = torch.empty(m, n, device="cuda", dtype=torch.float32 if args.f32_out else torch.bfloat16)
         fn = lambda: ops.linear(ctx, x, w, out)

@@ -34,6 +34,7 @@ def main(argv: list[str] | None = None) -> int:
         "--max-tokens", required=True, type=int,
         help="most tokens live requests hold at any time (each request rounded up to a multiple of 64)",
     )
+    parser.add_argument("--max-requests", type=int, default=4, help="most requests live at any time: the per-request state slots made (default 4)")
     parser.add_argument("--page-size", type=int, default=DEFAULT_PAGE_SIZE, help="tokens per cache page (divides 64)")
     parser.add_argument("--device", default="cuda:0")
     parser.add_argument(
@@ -44,6 +45,8 @@ def main(argv: list[str] | None = None) -> int:
     args = parser.parse_args(argv)
     if args.max_tokens <= 0:
         parser.error("--max-tokens must be positive")
+    if args.max_requests <= 0:
+        parser.error("--max-requests must be positive")
     if args.page_size <= 0 or 64 % args.page_size:
         parser.error("--page-size must divide 64")
 
@@ -66,7 +69,7 @@ def main(argv: list[str] | None = None) -> int:
         dtype=model.dtype,
         device=model.device,
         page_size=args.page_size,
-        max_num_sequences=max(4, pool_tokens // 64),
+        max_num_sequences=args.max_requests,
         max_model_length=min(config.max_position_embeddings, pool_tokens),
         step_tokens=pool_tokens,
         num_pages=pool_tokens // args.page_size,

@@ -3,6 +3,7 @@ from .gunedra_config import GunedraConfig
 from .lerorax_config import LeroraxConfig
 from .zetizen_config import ZetizenConfig
 from .model_config import ConfigError, ModelConfig, Qwen2Config, read_config_json
+from .tosipel_config import TosipelConfig
 from .registry import (
     Architecture,
     parse_config,
@@ -19,6 +20,7 @@ __all__ = [
     "LeroraxConfig",
     "ModelConfig",
     "Qwen2Config",
+    "TosipelConfig",
     "ZetizenConfig",
     "parse_config",
     "read_config_json",

@@ -27,31 +27,9 @@ import math
 from dataclasses import dataclass, field
 from typing import Any, ClassVar
 
-from .model_config import ConfigError, ModelConfig, _take
+from .model_config import ConfigError, ModelConfig, _number, _object, _positive, _take
 
 MIXER_TYPES = ("attention", "parallel")
-
-
-def _object(raw: dict, key: str, where: str, optional: bool = False) -> dict | None:
-    value = raw.get(key)
-    if value is None and optional:
-        return None
-    if not isinstance(value, dict):
-        raise ConfigError(f"{where}.{key} must be an object")
-    return value
-
-
-def _positive(raw: dict, keys: tuple[str, ...], where: str) -> None:
-    for key in keys:
-        if _take(raw, key, int) <= 0:
-            raise ConfigError(f"{where}.{key} must be positive")
-
-
-def _number(raw: dict, key: str, where: str, *, above: float | None = None) -> float:
-    value = _take(raw, key, float)
-    if not math.isfinite(value) or (above is not None and not value > above):
-        raise ConfigError(f"{where}.{key}={value} must be finite" + ("" if above is None else f" and above {above}"))
-    return value
 
 
 @dataclass(frozen=True)

@@ -22,6 +22,8 @@
 // window key > position - window. Behind a window the first `keep_first` keys of a request may
 // stay visible (FORM_KEPT): the walk takes their tiles first, then the window's. FORM_SIGMOID turns
 // a score into a weight by a sigmoid instead of a softmax: no maximum, no sum, no rescaling.
+// A sink (any softmax form) is the start of a row's running maximum and sum, (sink, 1), in the
+// one warp and split that owns the row's first keys.
 #include <cuda.h>
 
 #include <type_traits>
@@ -463,6 +465,11 @@ paged_flash_attention_kernel(const FlashParams p) {
   float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
   const float gate0 = SIGMOID && live0 ? __ldg(p.shape.sigmoid_bias + head0) * kLog2e : 0.f;
   const float gate1 = SIGMOID && live1 ? __ldg(p.shape.sigmoid_bias + head1) * kLog2e : 0.f;
+  if (!SIGMOID && p.shape.sink != nullptr && (!DECODE || (warp == 0 && split == 0))) {
+    // the row's sum is spread over four lanes: one of them holds the sink's term
+    if (live0) m0 = __ldg(p.shape.sink + head0) * kLog2e, l0 = (lane & 3) == 0 ? 1.f : 0.f;
+    if (live1) m1 = __ldg(p.shape.sink + head1) * kLog2e, l1 = (lane & 3) == 0 ? 1.f : 0.f;
+  }
 
   // Fill the ring. Tiles that hold only keys of earlier steps are requested before the wait
   // for the kernel in front (decode only); they always come first in the block's range. Every
@@ -927,6 +934,10 @@ paged_decode_tma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_
   const int mi = lane >> 3;
   const float gate0 = SIGMOID && live0 ? __ldg(p.shape.sigmoid_bias + kv_head * p.group + r0) * kLog2e : 0.f;
   const float gate1 = SIGMOID && live1 ? __ldg(p.shape.sigmoid_bias + kv_head * p.group + r1) * kLog2e : 0.f;
+  if (!SIGMOID && p.shape.sink != nullptr && warp == 0 && split == 0) {
+    if (live0) m0 = __ldg(p.shape.sink + kv_head * p.group + r0) * kLog2e, l0 = (lane & 3) == 0 ? 1.f : 0.f;
+    if (live1) m1 = __ldg(p.shape.sink + kv_head * p.group + r1) * kLog2e, l1 = (lane & 3) == 0 ? 1.f : 0.f;
+  }
 
   for (int j = 0; j < mine; ++j) {
     const int slot = j % stages;
@@ -1178,8 +1189,9 @@ B200_API int b200_paged_flash_attention(const void* q, const void* k_arena, cons
                                         int num_pages, int q_heads, int kv_heads, int head_dim,
                                         int page_size, int window, int keep_first, float scale, int decode, int splits,
                                         int value_head, float softcap, const float* bias, int bias_reach, int chunk,
-                                        const float* sigmoid_bias, float* scratch, int* err, cudaStream_t stream) {
+                                        const float* sigmoid_bias, const float* sink, float* scratch, int* err, cudaStream_t stream) {
   if (num_seqs == 0) return 0;
+  B200_REQUIRE(sigmoid_bias == nullptr || sink == nullptr, "paged_flash_attention: a sink is a term of a softmax, sigmoid weights have none");
   B200_REQUIRE(softcap >= 0.f && chunk >= 0 && (bias == nullptr || bias_reach >= 0), "paged_flash_attention: bad score shape");
   const bool shaped = softcap > 0.f || bias != nullptr || chunk > 0;
   B200_REQUIRE(keep_first >= 0 && !(shaped && (sigmoid_bias != nullptr || (window > 0 && keep_first > 0))),
@@ -1222,7 +1234,7 @@ B200_API int b200_paged_flash_attention(const void* q, const void* k_arena, cons
   p.plane_tokens = every_value_head ? tokens : 0;
   p.scale_log2 = scale * kLog2e;
   p.scale = scale;
-  p.shape = ScoreShape{softcap, bias, bias_reach, chunk, sigmoid_bias};
+  p.shape = ScoreShape{softcap, bias, bias_reach, chunk, sigmoid_bias, sink};
   p.cap_twice_inv = softcap > 0.f ? 2.f / softcap : 0.f;
   p.err = err;
   p.partial_out = scratch;
@@ -1261,8 +1273,9 @@ B200_API int b200_paged_decode_attention_tma(const void* q, const void* k_arena,
                                              const int* seq_kv_len, int num_seqs, int max_pages, int num_pages,
                                              int q_heads, int kv_heads, int head_dim, int page_size, int window,
                                              int keep_first, float scale, int splits, int stages,
-                                             const float* sigmoid_bias, float* scratch, int* err, cudaStream_t stream) {
+                                             const float* sigmoid_bias, const float* sink, float* scratch, int* err, cudaStream_t stream) {
   if (num_seqs == 0) return 0;
+  B200_REQUIRE(sigmoid_bias == nullptr || sink == nullptr, "decode attention (TMA): a sink is a term of a softmax, sigmoid weights have none");
   B200_REQUIRE(b200_decode_attention_tma_supported(q_heads, kv_heads, head_dim, page_size),
                "decode attention (TMA): unsupported shape (heads %d/%d, head_dim %d, page %d)", q_heads, kv_heads,
                head_dim, page_size);
@@ -1299,7 +1312,7 @@ B200_API int b200_paged_decode_attention_tma(const void* q, const void* k_arena,
   p.plane_tokens = 0;
   p.scale_log2 = scale * kLog2e;
   p.scale = scale;
-  p.shape = ScoreShape{0.f, nullptr, 0, 0, sigmoid_bias};
+  p.shape = ScoreShape{0.f, nullptr, 0, 0, sigmoid_bias, sink};
   p.cap_twice_inv = 0.f;
   p.err = err;
   p.partial_out = scratch;

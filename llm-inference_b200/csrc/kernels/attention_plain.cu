@@ -13,7 +13,8 @@
 // learned bias by the key's distance, read from a table [q_heads][reach + 1] at min(pos - key, reach) and added after
 // the cap; and restricted to the query's own chunk of positions, keys from floor(pos / chunk) * chunk on. With
 // `sigmoid_bias` a visible key weighs sigmoid(score + bias of the head) and nothing is normalised. With a window the
-// first `keep_first` keys of the request stay visible in front of it.
+// first `keep_first` keys of the request stay visible in front of it. With `sink` the running maximum and sum start at
+// (sink of the head, 1): a term exp(sink) of the denominator that has no key and no value.
 #include "common.cuh"
 
 namespace {
@@ -83,7 +84,7 @@ paged_attention_plain_kernel(const T* __restrict__ q, const T* __restrict__ k_ar
   float acc[kMaxDimsPerThread];
 #pragma unroll
   for (int i = 0; i < kMaxDimsPerThread; ++i) acc[i] = 0.f;
-  float running_max = -INFINITY, running_sum = 0.f;
+  float running_max = shape.sink ? shape.sink[h] : -INFINITY, running_sum = shape.sink ? 1.f : 0.f;
 
   // The walk counts visible keys: the kept ones in front of the window, then lo .. pos.
   const int kept = window > 0 ? min(keep_first, lo) : 0;
@@ -148,10 +149,11 @@ B200_API int b200_paged_attention_plain(const void* q, const void* k_arena, cons
                                         void* out, int tokens, int q_heads, int kv_heads,
                                         int head_dim, int page_size, int window, int keep_first, float scale,
                                         int value_head, float softcap, const float* bias, int bias_reach, int chunk,
-                                        const float* sigmoid_bias, int dtype, int* err, cudaStream_t stream) {
+                                        const float* sigmoid_bias, const float* sink, int dtype, int* err, cudaStream_t stream) {
   if (tokens == 0) return 0;
   B200_REQUIRE(softcap >= 0.f && chunk >= 0 && (bias == nullptr || bias_reach >= 0), "paged_attention_plain: bad score shape");
-  const ScoreShape shape{softcap, bias, bias_reach, chunk, sigmoid_bias};
+  B200_REQUIRE(sigmoid_bias == nullptr || sink == nullptr, "paged_attention_plain: a sink is a term of a softmax, sigmoid weights have none");
+  const ScoreShape shape{softcap, bias, bias_reach, chunk, sigmoid_bias, sink};
   B200_REQUIRE(tokens > 0 && q_heads > 0 && kv_heads > 0 && q_heads % kv_heads == 0,
                "paged_attention_plain: %d query heads over %d kv heads", q_heads, kv_heads);
   B200_REQUIRE(head_dim > 0 && head_dim % 8 == 0 && head_dim <= kThreads * kMaxDimsPerThread,

@@ -16,7 +16,8 @@
 // python/instinct/batches.py:110-113: key <= query position and, with a window,
 // key > position - window. Behind a window the first `keep_first` keys of a request may stay
 // visible (KEPT): the walk takes their tiles first, then the window's. SIGMOID turns a score into
-// a weight by a sigmoid: no maximum, no sum, nothing the two softmax groups have to agree on.
+// a weight by a sigmoid: no maximum, no sum, nothing the two softmax groups have to agree on. A
+// sink (the softmax forms) is one more term of a row's sum, added when the row is finished.
 //
 // Every wait (mbarriers, and the shared-memory word the two softmax threads of a row pass the
 // turn with) is bounded; on a timeout the block records ERRBIT_TIMEOUT, skips its further waits,
@@ -59,6 +60,7 @@ struct PrefillParams {
   int window;
   int keep_first;  // the KEPT and SIGMOID forms only: the first this many keys stay visible in front of the window
   const float* sigmoid_bias;  // [q_heads], the SIGMOID form only
+  const float* sink;          // [q_heads] or null, the softmax forms only
   int value_head;  // >= 0: every block takes its values from this kv head's rows of the pages (keys stay its own)
   float scale_log2;
   // The capped form only: scores pass cap * tanh(score / cap) and a query sees only the keys of its own chunk.
@@ -684,13 +686,13 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap k_map, const __
       l = 1.f;  // nothing is normalised
     } else {
       if (!turn_of(num_tiles)) ok = false;
-      {
-        const float m = *shared_m;
-        if (m != seen) l *= seen == -INFINITY ? 0.f : exp2f(seen - m);
-      }
+      const float m = *shared_m;
+      if (m != seen) l *= seen == -INFINITY ? 0.f : exp2f(seen - m);
       row_l[group][r] = l;
       asm volatile("bar.sync 1, %0;" ::"n"(kSoftmaxThreads) : "memory");
       l = row_l[0][r] + row_l[1][r];
+      // The sink's term against the same offset (an overflow means that the keys weigh nothing beside it: 1 / l is zero).
+      if (p.sink != nullptr && live) l += exp2f(__ldg(p.sink + q_head) * kLog2eA - m);
     }
     if (ok && num_tiles > 0) ok = bar_wait(&o_done[(num_tiles - 1) & 3], ((num_tiles - 1) >> 2) & 1);
     if (!ok && lane == 0) atomicOr(p.err, ERRBIT_TIMEOUT_A);
@@ -781,9 +783,10 @@ B200_API int b200_flash_prefill_tcgen05(const void* q, const void* k_arena, cons
                                         int max_kv_len, int max_pages, int num_pages, int q_heads, int kv_heads,
                                         int head_dim, int page_size, int window, int keep_first, float scale, int value_head,
                                         float softcap, const float* bias, const float* bias_peak, int bias_reach, int chunk,
-                                        const float* sigmoid_bias, int* err, cudaStream_t stream) {
+                                        const float* sigmoid_bias, const float* sink, int* err, cudaStream_t stream) {
   if (num_seqs == 0) return 0;
   B200_REQUIRE(softcap >= 0.f && chunk >= 0, "flash_prefill_tcgen05: bad cap or chunk");
+  B200_REQUIRE(sigmoid_bias == nullptr || sink == nullptr, "flash_prefill_tcgen05: a sink is a term of a softmax, sigmoid weights have none");
   B200_REQUIRE(bias == nullptr || (bias_peak != nullptr && bias_reach >= 0), "flash_prefill_tcgen05: a bias by distance comes with its rows' maxima");
   B200_REQUIRE(b200_flash_prefill_tcgen05_supported(q_heads, kv_heads, head_dim, page_size, max_kv_len),
                "flash_prefill_tcgen05: unsupported shape (heads %d/%d, head_dim %d, page %d, %d keys)", q_heads, kv_heads,
@@ -812,6 +815,7 @@ B200_API int b200_flash_prefill_tcgen05(const void* q, const void* k_arena, cons
   p.window = window;
   p.keep_first = keep_first;
   p.sigmoid_bias = sigmoid_bias;
+  p.sink = sink;
   p.value_head = value_head;
   p.scale_log2 = scale * kLog2eA;
   p.scale = scale;

@@ -208,8 +208,18 @@ __device__ __forceinline__ float block_max(float v, float* scratch) {
   return total;
 }
 
+// The gated units of the feed-forwards: silu(gate) * up, or gelu(gate) * up with the tanh form of gelu,
+// 0.5 g (1 + tanh(y)) = g / (1 + e^(-2 y)) with y = sqrt(2 / pi) (g + 0.044715 g^3).
+template <bool GELU>
+__device__ __forceinline__ float gated_unit(float gate, float up) {
+  constexpr float kTwiceRoot = 1.5957691216057308f;  // 2 sqrt(2 / pi)
+  const float slope = GELU ? kTwiceRoot * fmaf(0.044715f * gate * gate, gate, gate) : gate;
+  return gate / (1.f + expf(-slope)) * up;
+}
+
 // What an attention kernel does to a score beyond the scale: a soft cap, a learned bias by the key's distance and a
-// restriction to the query's own chunk of positions; and how a score becomes a weight (softmax, or a sigmoid per key).
+// restriction to the query's own chunk of positions; and how a score becomes a weight (softmax, with or without a sink, or
+// a sigmoid per key).
 // All zero / null: nothing, and a softmax.
 struct ScoreShape {
   float softcap;      // > 0: s <- softcap * tanh(s / softcap)
@@ -217,6 +227,7 @@ struct ScoreShape {
   int bias_reach;
   int chunk;          // > 0: a query at `pos` sees keys from floor(pos / chunk) * chunk on only
   const float* sigmoid_bias;  // [q_heads]: a visible key weighs sigmoid(score + bias of the head), nothing is normalised; null: softmax
+  const float* sink;  // [q_heads]: the softmax's denominator also holds exp(sink of the head), not scaled, without a value; null: none
 };
 
 // `s` is the scaled score, `bias_row` the query head's row of the bias table (or null), `distance` = pos - key >= 0.

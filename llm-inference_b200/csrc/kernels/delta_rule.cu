@@ -6,9 +6,12 @@
 // q and k are unit vectors per head (q also times dk^-1/2) made from projections that first pass
 // a short causal convolution over time and silu; g = exp(-exp(A_log[h]) softplus(a + dt_bias));
 // beta = sigmoid(b). The state and the convolution's last taps - 1 inputs live in per-request
-// slots. Everything that enters the recurrence is 32-bit.
+// slots. Everything that enters the recurrence is 32-bit. The form with one decay per head has a
+// recurrence of its own (delta_head.cu); `delta_prepare` and `delta_output` serve both, the latter
+// with a sigmoid or a silu of the gate.
 //
-// Kernels: `delta_prepare` (one block per token: convolution, silu, unit vectors, beta, decay),
+// Kernels: `delta_prepare` (one block per token: convolution, silu, unit vectors, beta, decay,
+// and k . q where the recurrence wants it),
 // `conv_state_update` (one block per request: the slot's last inputs), `delta_recurrence` (the
 // columns of S are independent, so a thread group owns a column and walks the request's tokens),
 // `delta_output` (o / rms(o) * w * sigmoid(gate)).
@@ -22,14 +25,16 @@ __device__ __forceinline__ float softplus_f(float x) { return x > 20.f ? x : log
 // `proj` rows: [q (kv_heads*dk) | k (kv_heads*dk) | v (heads*dv) | b (heads)]; the first
 // `channels` = 2 kv_heads dk + heads dv columns pass the convolution. `conv_state`
 // [slots][taps-1][channels] holds each request's last inputs, oldest first. `decay_in`
-// [tokens][heads*dk] is W_a2 W_a1 h.
+// [tokens][heads * span] is the projection the decays come from. Without `kq_out` there is a decay per head and key
+// channel (span = dk) and `decay_out` takes the factors; with it there is one per head (span = 1), `decay_out` takes
+// their logarithms, and `kq_out` k . q per kv head, of the vectors as they are written.
 template <typename T>
 __global__ void delta_prepare_kernel(const T* proj, int ld, const T* decay_in, int decay_ld,
                                      const float* __restrict__ taps_w, int taps, const T* conv_state,
                                      const float* __restrict__ a_log, const float* __restrict__ dt_bias,
                                      const int* token_seq, const int* seq_q_start, const int* seq_slot, int heads,
                                      int kv_heads, int dk, int dv, float* q_out, float* k_out, float* v_out, float* beta_out,
-                                     float* decay_out) {
+                                     float* decay_out, float* kq_out) {
   extern __shared__ float y[];  // [channels]
   wait_for_predecessor();
   let_successor_start();
@@ -51,7 +56,7 @@ __global__ void delta_prepare_kernel(const T* proj, int ld, const T* decay_in, i
   }
   __syncthreads();
   const int lane = tid & 31, warp = tid >> 5, warps = blockDim.x >> 5;
-  // unit vectors: one warp per (q or k, kv head)
+  // unit vectors: one warp per (q or k, kv head); k . q is worked out beside k
   for (int item = warp; item < 2 * kv_heads; item += warps) {
     const float* src = y + item * dk;
     float ss = 0.f;
@@ -59,15 +64,28 @@ __global__ void delta_prepare_kernel(const T* proj, int ld, const T* decay_in, i
     ss = warp_sum(ss);
     const bool is_q = item < kv_heads;
     const float factor = (1.f / sqrtf(ss + 1e-6f)) * (is_q ? 1.f / sqrtf(static_cast<float>(dk)) : 1.f);
-    float* dst = (is_q ? q_out : k_out) + static_cast<int64_t>(t) * qk + (is_q ? item : item - kv_heads) * dk;
+    const int head = is_q ? item : item - kv_heads;
+    float* dst = (is_q ? q_out : k_out) + static_cast<int64_t>(t) * qk + head * dk;
     for (int i = lane; i < dk; i += 32) dst[i] = src[i] * factor;
+    if (kq_out != nullptr && !is_q) {
+      const float* q = y + head * dk;
+      float q_ss = 0.f, dot = 0.f;
+      for (int i = lane; i < dk; i += 32) q_ss = fmaf(q[i], q[i], q_ss), dot = fmaf(q[i], src[i], dot);
+      q_ss = warp_sum(q_ss);
+      dot = warp_sum(dot);
+      if (lane == 0)
+        kq_out[static_cast<int64_t>(t) * kv_heads + head] = dot * factor * ((1.f / sqrtf(q_ss + 1e-6f)) * (1.f / sqrtf(static_cast<float>(dk))));
+    }
   }
   for (int i = tid; i < vw; i += blockDim.x) v_out[static_cast<int64_t>(t) * vw + i] = y[2 * qk + i];
   for (int h = tid; h < heads; h += blockDim.x)
     beta_out[static_cast<int64_t>(t) * heads + h] = sigmoid_f(to_f32<T>(proj[static_cast<int64_t>(t) * ld + channels + h]));
-  for (int i = tid; i < heads * dk; i += blockDim.x) {
+  const bool per_head = kq_out != nullptr;
+  const int span = per_head ? 1 : dk;
+  for (int i = tid; i < heads * span; i += blockDim.x) {
     const float step = softplus_f(to_f32<T>(decay_in[static_cast<int64_t>(t) * decay_ld + i]) + dt_bias[i]);
-    decay_out[static_cast<int64_t>(t) * heads * dk + i] = expf(-expf(a_log[i / dk]) * step);
+    const float log_decay = -expf(a_log[i / span]) * step;
+    decay_out[static_cast<int64_t>(t) * heads * span + i] = per_head ? log_decay : expf(log_decay);
   }
 }
 
@@ -221,8 +239,8 @@ delta_recurrence_kernel(const float* q, const float* k, const float* v, const fl
   }
 }
 
-// out[t, h, :] = o / rms(o) * w * sigmoid(gate[t, h, :]); one warp per (token, head).
-template <typename T>
+// out[t, h, :] = o / rms(o) * w * sigmoid(gate[t, h, :]), or silu of the gate; one warp per (token, head).
+template <typename T, bool SILU>
 __global__ void delta_output_kernel(const float* o, const float* __restrict__ weight, const T* gate, int gate_ld, int rows,
                                     int heads, int dv, float eps, T* out) {
   wait_for_predecessor();
@@ -238,7 +256,10 @@ __global__ void delta_output_kernel(const float* o, const float* __restrict__ we
   const float inv = 1.f / sqrtf(ss / static_cast<float>(dv) + eps);
   const T* g = gate + static_cast<int64_t>(t) * gate_ld + h * dv;
   T* dst = out + static_cast<int64_t>(item) * dv;
-  for (int i = lane; i < dv; i += 32) dst[i] = from_f32<T>(src[i] * inv * weight[i] * sigmoid_f(to_f32<T>(g[i])));
+  for (int i = lane; i < dv; i += 32) {
+    const float x = to_f32<T>(g[i]);
+    dst[i] = from_f32<T>(src[i] * inv * weight[i] * (SILU ? x * sigmoid_f(x) : sigmoid_f(x)));
+  }
 }
 
 }  // namespace
@@ -247,7 +268,7 @@ B200_API int b200_delta_prepare(const void* proj, int ld, const void* decay_in, 
                                 void* conv_state, const float* a_log, const float* dt_bias, const int* token_seq,
                                 const int* seq_q_start, const int* seq_q_len, const int* seq_slot, int tokens, int seqs,
                                 int heads, int kv_heads, int dk, int dv, float* q_out, float* k_out, float* v_out,
-                                float* beta_out, float* decay_out, int dtype, cudaStream_t stream) {
+                                float* beta_out, float* decay_out, float* kq_out, int dtype, cudaStream_t stream) {
   if (tokens == 0) return 0;
   B200_REQUIRE(tokens > 0 && seqs > 0 && heads > 0 && kv_heads > 0 && heads % kv_heads == 0 && dk > 0 && dv > 0 && taps >= 1,
                "delta_prepare: bad sizes");
@@ -260,7 +281,7 @@ B200_API int b200_delta_prepare(const void* proj, int ld, const void* decay_in, 
       cudaFuncSetAttribute(delta_prepare_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
     launch_kernel(delta_prepare_kernel<float>, dim3(tokens), dim3(threads), smem, stream, static_cast<const float*>(proj), ld,
                   static_cast<const float*>(decay_in), decay_ld, taps_w, taps, static_cast<const float*>(conv_state), a_log,
-                  dt_bias, token_seq, seq_q_start, seq_slot, heads, kv_heads, dk, dv, q_out, k_out, v_out, beta_out, decay_out);
+                  dt_bias, token_seq, seq_q_start, seq_slot, heads, kv_heads, dk, dv, q_out, k_out, v_out, beta_out, decay_out, kq_out);
     if (int status = b200_check_launch("delta_prepare")) return status;
     launch_kernel(conv_state_update_kernel<float>, dim3(seqs), dim3(threads), 0, stream, static_cast<const float*>(proj), ld,
                   channels, taps, seq_q_start, seq_q_len, seq_slot, static_cast<float*>(conv_state));
@@ -271,7 +292,7 @@ B200_API int b200_delta_prepare(const void* proj, int ld, const void* decay_in, 
     launch_kernel(delta_prepare_kernel<__nv_bfloat16>, dim3(tokens), dim3(threads), smem, stream,
                   static_cast<const __nv_bfloat16*>(proj), ld, static_cast<const __nv_bfloat16*>(decay_in), decay_ld, taps_w,
                   taps, static_cast<const __nv_bfloat16*>(conv_state), a_log, dt_bias, token_seq, seq_q_start, seq_slot, heads,
-                  kv_heads, dk, dv, q_out, k_out, v_out, beta_out, decay_out);
+                  kv_heads, dk, dv, q_out, k_out, v_out, beta_out, decay_out, kq_out);
     if (int status = b200_check_launch("delta_prepare")) return status;
     launch_kernel(conv_state_update_kernel<__nv_bfloat16>, dim3(seqs), dim3(threads), 0, stream,
                   static_cast<const __nv_bfloat16*>(proj), ld, channels, taps, seq_q_start, seq_q_len, seq_slot,
@@ -321,18 +342,18 @@ B200_API int b200_delta_recurrence(const float* q, const float* k, const float* 
 }
 
 B200_API int b200_delta_output(const float* o, const float* weight, const void* gate, int gate_ld, int rows, int heads, int dv,
-                               float eps, void* out, int dtype, cudaStream_t stream) {
+                               float eps, int silu, void* out, int dtype, cudaStream_t stream) {
   if (rows == 0) return 0;
   B200_REQUIRE(rows > 0 && heads > 0 && dv > 0, "delta_output: bad sizes");
   const int threads = 128;
   const int64_t items = static_cast<int64_t>(rows) * heads;
   const unsigned blocks = static_cast<unsigned>((items + 3) / 4);
   if (dtype == DTYPE_F32) {
-    launch_kernel(delta_output_kernel<float>, dim3(blocks), dim3(threads), 0, stream, o, weight, static_cast<const float*>(gate),
-                  gate_ld, rows, heads, dv, eps, static_cast<float*>(out));
+    launch_kernel(silu ? delta_output_kernel<float, true> : delta_output_kernel<float, false>, dim3(blocks), dim3(threads), 0, stream, o, weight,
+                  static_cast<const float*>(gate), gate_ld, rows, heads, dv, eps, static_cast<float*>(out));
   } else if (dtype == DTYPE_BF16) {
-    launch_kernel(delta_output_kernel<__nv_bfloat16>, dim3(blocks), dim3(threads), 0, stream, o, weight,
-                  static_cast<const __nv_bfloat16*>(gate), gate_ld, rows, heads, dv, eps, static_cast<__nv_bfloat16*>(out));
+    launch_kernel(silu ? delta_output_kernel<__nv_bfloat16, true> : delta_output_kernel<__nv_bfloat16, false>, dim3(blocks), dim3(threads), 0, stream,
+                  o, weight, static_cast<const __nv_bfloat16*>(gate), gate_ld, rows, heads, dv, eps, static_cast<__nv_bfloat16*>(out));
   } else {
     return b200_fail("delta_output: unknown dtype %d", dtype);
   }

@@ -233,19 +233,21 @@ B200_API int b200_rmsnorm(float* x, const void* delta, const float* weight, void
 // (python/instinct/backends/dense.py:124-128; cuda/kernels.cu:100-106). The input row holds
 // gate and up interleaved: gu[t, 2i] is gate_i and gu[t, 2i + 1] is up_i, which is how the
 // feed-forward stores its fused gate/up matrix.
-template <typename T>
-__global__ void silu_mul_kernel(const T* gu, T* out, int64_t total) {
+// With GELU the gate passes the tanh form of gelu instead of silu.
+template <typename T, bool GELU>
+__global__ void gated_mul_kernel(const T* gu, T* out, int64_t total) {
   wait_for_predecessor();
   let_successor_start();
   const int64_t idx = static_cast<int64_t>(blockIdx.x) * blockDim.x + threadIdx.x;
   if (idx >= total) return;
   const float g = to_f32<T>(gu[2 * idx]);
   const float u = to_f32<T>(gu[2 * idx + 1]);
-  out[idx] = from_f32<T>(g / (1.f + expf(-g)) * u);
+  out[idx] = from_f32<T>(gated_unit<GELU>(g, u));
 }
 
 // bfloat16, eight outputs per thread: two 16-byte loads, one 16-byte store.
-__global__ void silu_mul_bf16x8_kernel(const __nv_bfloat16* gu, __nv_bfloat16* out,
+template <bool GELU>
+__global__ void gated_mul_bf16x8_kernel(const __nv_bfloat16* gu, __nv_bfloat16* out,
                                        int64_t groups) {
   wait_for_predecessor();
   let_successor_start();
@@ -260,21 +262,21 @@ __global__ void silu_mul_bf16x8_kernel(const __nv_bfloat16* gu, __nv_bfloat16* o
   for (int i = 0; i < 4; ++i) {
     const float2 p = __bfloat1622float2(a[i]);
     const float2 q = __bfloat1622float2(b[i]);
-    r[i] = __float2bfloat16_rn(p.x / (1.f + expf(-p.x)) * p.y);
-    r[4 + i] = __float2bfloat16_rn(q.x / (1.f + expf(-q.x)) * q.y);
+    r[i] = __float2bfloat16_rn(gated_unit<GELU>(p.x, p.y));
+    r[4 + i] = __float2bfloat16_rn(gated_unit<GELU>(q.x, q.y));
   }
   reinterpret_cast<uint4*>(out)[idx] = *reinterpret_cast<const uint4*>(r);
 }
 
-B200_API int b200_silu_mul(const void* gate_up, void* out, int tokens, int inter, int dtype,
-                           cudaStream_t stream) {
+template <bool GELU>
+static int gated_mul(const char* name, const void* gate_up, void* out, int tokens, int inter, int dtype, cudaStream_t stream) {
   if (tokens == 0) return 0;
-  B200_REQUIRE(tokens > 0 && inter > 0, "silu_mul: bad sizes");
+  B200_REQUIRE(tokens > 0 && inter > 0, "%s: bad sizes", name);
   const int64_t total = static_cast<int64_t>(tokens) * inter;
   const int threads = 256;
   if (dtype == DTYPE_F32) {
     const unsigned blocks = static_cast<unsigned>((total + threads - 1) / threads);
-    launch_kernel(silu_mul_kernel<float>, dim3(blocks), dim3(threads), 0, stream,
+    launch_kernel(gated_mul_kernel<float, GELU>, dim3(blocks), dim3(threads), 0, stream,
                   static_cast<const float*>(gate_up), static_cast<float*>(out), total);
   } else if (dtype == DTYPE_BF16) {
     const bool vec = total % 8 == 0 && reinterpret_cast<uintptr_t>(gate_up) % 16 == 0 &&
@@ -282,15 +284,23 @@ B200_API int b200_silu_mul(const void* gate_up, void* out, int tokens, int inter
     if (vec) {
       const int64_t groups = total / 8;
       const unsigned blocks = static_cast<unsigned>((groups + threads - 1) / threads);
-      launch_kernel(silu_mul_bf16x8_kernel, dim3(blocks), dim3(threads), 0, stream,
+      launch_kernel(gated_mul_bf16x8_kernel<GELU>, dim3(blocks), dim3(threads), 0, stream,
                     static_cast<const __nv_bfloat16*>(gate_up), static_cast<__nv_bfloat16*>(out), groups);
     } else {
       const unsigned blocks = static_cast<unsigned>((total + threads - 1) / threads);
-      launch_kernel(silu_mul_kernel<__nv_bfloat16>, dim3(blocks), dim3(threads), 0, stream,
+      launch_kernel(gated_mul_kernel<__nv_bfloat16, GELU>, dim3(blocks), dim3(threads), 0, stream,
                     static_cast<const __nv_bfloat16*>(gate_up), static_cast<__nv_bfloat16*>(out), total);
     }
   } else {
-    return b200_fail("silu_mul: unknown dtype %d", dtype);
+    return b200_fail("%s: unknown dtype %d", name, dtype);
   }
-  return b200_check_launch("silu_mul");
+  return b200_check_launch(name);
+}
+
+B200_API int b200_silu_mul(const void* gate_up, void* out, int tokens, int inter, int dtype, cudaStream_t stream) {
+  return gated_mul<false>("silu_mul", gate_up, out, tokens, inter, dtype, stream);
+}
+
+B200_API int b200_gelu_mul(const void* gate_up, void* out, int tokens, int inter, int dtype, cudaStream_t stream) {
+  return gated_mul<true>("gelu_mul", gate_up, out, tokens, inter, dtype, stream);
 }

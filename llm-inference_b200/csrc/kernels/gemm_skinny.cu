@@ -19,8 +19,8 @@
 // W stored [out, in] (python/instinct/backends/base.py:83-101); the reference sends them to
 // cuBLASLt (cuda/execution_context.cu:95-110).
 //
-// Epilogues: bfloat16 or float32 rows of Y, or SwiGLU over interleaved rows of W (row 2j is
-// gate_j, row 2j + 1 is up_j): out[m, j] = silu(y[m, 2j]) * y[m, 2j + 1]
+// Epilogues: bfloat16 or float32 rows of Y, or a gated unit over interleaved rows of W (row 2j is
+// gate_j, row 2j + 1 is up_j): out[m, j] = silu(y[m, 2j]) * y[m, 2j + 1], or gelu for silu
 // (python/instinct/backends/dense.py:124-128).
 #include "common.cuh"
 
@@ -36,7 +36,8 @@ struct SkinnyStages {
   static constexpr int value = MT == 1 ? 12 : 8;
 };
 
-enum : int { EPI_BF16 = 0, EPI_F32 = 1, EPI_SWIGLU = 2, EPI_SQUARED_RELU = 3 };
+enum : int { EPI_BF16 = 0, EPI_F32 = 1, EPI_SWIGLU = 2, EPI_SQUARED_RELU = 3, EPI_GEGLU = 4 };
+__host__ __device__ constexpr bool gated(int epi) { return epi == EPI_SWIGLU || epi == EPI_GEGLU; }  // rows of W come in gate/up pairs
 
 __device__ __forceinline__ void mma_bf16_16816(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2,
                                                uint32_t a3, uint32_t b0, uint32_t b1) {
@@ -233,7 +234,7 @@ skinny_gemm_kernel(const __nv_bfloat16* __restrict__ W, const __nv_bfloat16* X,
     }
     return;
   }
-  if constexpr (EPI == EPI_SWIGLU) {
+  if constexpr (gated(EPI)) {
     const int pairs = block_rows / 2;
     for (int item = threadIdx.x; item < M * pairs; item += kSkinnyThreads) {
       const int m = item / pairs, j = item - m * pairs;
@@ -241,7 +242,7 @@ skinny_gemm_kernel(const __nv_bfloat16* __restrict__ W, const __nv_bfloat16* X,
       if (n >= N) continue;
       const float gate = total(2 * j, m), up = total(2 * j + 1, m);
       static_cast<__nv_bfloat16*>(Y)[static_cast<int64_t>(m) * (N / 2) + n / 2] =
-          __float2bfloat16_rn(gate / (1.f + expf(-gate)) * up);
+          __float2bfloat16_rn(gated_unit<EPI == EPI_GEGLU>(gate, up));
     }
   } else {
     for (int item = threadIdx.x; item < M * block_rows; item += kSkinnyThreads) {
@@ -328,7 +329,9 @@ int launch_skinny(const __nv_bfloat16* W, const __nv_bfloat16* X, void* Y, int M
       return launch_skinny_epilogue<MT, EPI_F32>(W, X, Y, M, N, K, plan, scratch, counters, stream, ordered, fold);
     case EPI_SWIGLU:
       return launch_skinny_epilogue<MT, EPI_SWIGLU>(W, X, Y, M, N, K, plan, scratch, counters, stream, ordered, fold);
-    case EPI_SQUARED_RELU:  // not around a folded norm (the callers refuse that)
+    case EPI_GEGLU:
+      return launch_skinny_as<MT, EPI_GEGLU, false>(W, X, Y, M, N, K, plan, scratch, counters, stream, ordered, fold);
+    case EPI_SQUARED_RELU:  // these two not around a folded norm (the callers refuse that)
       return launch_skinny_as<MT, EPI_SQUARED_RELU, false>(W, X, Y, M, N, K, plan, scratch, counters, stream, ordered, fold);
     default:
       return launch_skinny_epilogue<MT, EPI_BF16>(W, X, Y, M, N, K, plan, scratch, counters, stream, ordered, fold);
@@ -340,10 +343,10 @@ int launch_skinny(const __nv_bfloat16* W, const __nv_bfloat16* X, void* Y, int M
 constexpr int kSkinnyMaxRows = 16;
 
 // Shapes the kernel takes: at most 16 rows, K a multiple of 8 (16-byte rows), 16-byte aligned
-// operands; for the SwiGLU epilogue N even.
+// operands; for the gated epilogues N even.
 B200_API int b200_skinny_gemm_supported(int M, int N, int K, int epilogue) {
   if (M < 1 || M > kSkinnyMaxRows || N < 1 || K < 8 || K % 8) return 0;
-  if (epilogue == EPI_SWIGLU && N % 2) return 0;
+  if (gated(epilogue) && N % 2) return 0;
   return 1;
 }
 
@@ -402,8 +405,8 @@ static int skinny_gemm_run(const void* W, const void* X, void* Y, int M, int N, 
                            int64_t scratch_floats, int* counters, int num_counters, const NormFold& fold,
                            cudaStream_t stream) {
   B200_REQUIRE(b200_skinny_gemm_supported(M, N, K, epilogue), "skinny_gemm: unsupported shape %d x %d x %d", M, N, K);
-  B200_REQUIRE(epilogue >= EPI_BF16 && epilogue <= EPI_SQUARED_RELU, "skinny_gemm: unknown epilogue %d", epilogue);
-  B200_REQUIRE(epilogue != EPI_SQUARED_RELU || (fold.ss_in == nullptr && fold.x == nullptr), "skinny_gemm: the squared relu has no folded form");
+  B200_REQUIRE(epilogue >= EPI_BF16 && epilogue <= EPI_GEGLU, "skinny_gemm: unknown epilogue %d", epilogue);
+  B200_REQUIRE(epilogue < EPI_SQUARED_RELU || (fold.ss_in == nullptr && fold.x == nullptr), "skinny_gemm: the squared relu and gelu epilogues have no folded form");
   B200_REQUIRE(reinterpret_cast<uintptr_t>(W) % 16 == 0 && reinterpret_cast<uintptr_t>(X) % 16 == 0,
                "skinny_gemm: operands must be 16-byte aligned");
   const SkinnyPlan plan = plan_skinny(N, K);
@@ -474,7 +477,7 @@ B200_API int b200_skinny_gemm_static(const void* W, const void* X, void* Y, int 
                                      cudaStream_t stream) {
   B200_REQUIRE(b200_skinny_gemm_supported(M, N, K, epilogue),
                "skinny_gemm_static: unsupported shape %d x %d x %d (at most 16 rows, K a multiple of 8)", M, N, K);
-  B200_REQUIRE(epilogue >= EPI_BF16 && epilogue <= EPI_SQUARED_RELU, "skinny_gemm_static: unknown epilogue %d", epilogue);
+  B200_REQUIRE(epilogue >= EPI_BF16 && epilogue <= EPI_GEGLU, "skinny_gemm_static: unknown epilogue %d", epilogue);
   B200_REQUIRE(W != nullptr && X != nullptr && Y != nullptr, "skinny_gemm_static: null operand");
   B200_REQUIRE(reinterpret_cast<uintptr_t>(W) % 16 == 0 && reinterpret_cast<uintptr_t>(X) % 16 == 0,
                "skinny_gemm_static: operands must be 16-byte aligned");

@@ -55,7 +55,8 @@ constexpr int kThreadsT = 192;   // warp 0: TMA, warp 1: MMA, warps 2-5: epilogu
 constexpr long long kWaitCycles = 4000000000LL;  // about two seconds
 constexpr int ERRBIT_TIMEOUT = 8;
 
-enum : int { EPI_BF16 = 0, EPI_F32 = 1, EPI_SWIGLU = 2, EPI_SQUARED_RELU = 3 };
+enum : int { EPI_BF16 = 0, EPI_F32 = 1, EPI_SWIGLU = 2, EPI_SQUARED_RELU = 3, EPI_GEGLU = 4 };
+__host__ __device__ constexpr bool gated(int epi) { return epi == EPI_SWIGLU || epi == EPI_GEGLU; }  // rows of W come in gate/up pairs
 
 __device__ __forceinline__ uint32_t smem_addr(const void* p) {
   return static_cast<uint32_t>(__cvta_generic_to_shared(p));
@@ -180,7 +181,7 @@ __device__ __forceinline__ void pull_slices_wide(const StreamParams& p, const fl
                                                  int rows, int r_begin, int n0) {
   const int columns = (rows + 3) / 4;
   const int total = columns * p.M;
-  constexpr bool swiglu = EPI == EPI_SWIGLU;
+  constexpr bool pairs_of_rows = gated(EPI);
   for (int base = tid; base < total; base += 128 * ITEMS) {
     float4 part[ITEMS][RANKS];
 #pragma unroll
@@ -208,12 +209,12 @@ __device__ __forceinline__ void pull_slices_wide(const StreamParams& p, const fl
       }
       const int n = n0 + r;
       const int live = min(4, min(r_begin + rows - r, p.N - n));  // rows of the item inside the slice and the matrix
-      if (swiglu) {
+      if (pairs_of_rows) {
 #pragma unroll
         for (int i = 0; i < 4; i += 2)
           if (i + 1 < live)
             static_cast<__nv_bfloat16*>(p.y)[static_cast<int64_t>(m) * (p.N / 2) + (n + i) / 2] =
-                __float2bfloat16_rn(values[i] / (1.f + expf(-values[i])) * values[i + 1]);
+                __float2bfloat16_rn(gated_unit<EPI == EPI_GEGLU>(values[i], values[i + 1]));
       } else {
 #pragma unroll
         for (int i = 0; i < 4; ++i)
@@ -228,7 +229,7 @@ __device__ __forceinline__ void pull_slices_wide(const StreamParams& p, const fl
 template <int EPI>
 __device__ __forceinline__ void pull_slices_narrow(const StreamParams& p, const float* partial, int members, int tid,
                                                    int rows, int r_begin, int n0) {
-  if constexpr (EPI == EPI_SWIGLU) {
+  if constexpr (gated(EPI)) {
     const int pairs = rows / 2;
     for (int item = tid; item < pairs * p.M; item += 128) {
       const int m = item / pairs, r = r_begin + 2 * (item - m * pairs);
@@ -251,7 +252,7 @@ __device__ __forceinline__ void pull_slices_narrow(const StreamParams& p, const 
       const int n = n0 + r;
       if (n < p.N)
         static_cast<__nv_bfloat16*>(p.y)[static_cast<int64_t>(m) * (p.N / 2) + n / 2] =
-            __float2bfloat16_rn(gate / (1.f + expf(-gate)) * up);
+            __float2bfloat16_rn(gated_unit<EPI == EPI_GEGLU>(gate, up));
     }
   } else {
     for (int item = tid; item < rows * p.M; item += 128) {
@@ -468,7 +469,7 @@ stream_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_const
           if (lane == 0 && m < kFoldTokens)
             p.fold.ss_out[(static_cast<int64_t>(blockIdx.x) * 4 + quarter) * kFoldTokens + m] = sq;
         }
-      } else if (EPI == EPI_SWIGLU) {
+      } else if (gated(EPI)) {
 #pragma unroll
         for (int i = 0; i < 16; ++i) {
           const int m = c0 + i;
@@ -476,7 +477,7 @@ stream_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_const
           const float up = __shfl_down_sync(0xffffffffu, gate, 1);
           if ((lane & 1) == 0 && m < p.M && n < p.N)
             static_cast<__nv_bfloat16*>(p.y)[static_cast<int64_t>(m) * (p.N / 2) + n / 2] =
-                __float2bfloat16_rn(gate / (1.f + expf(-gate)) * up);
+                __float2bfloat16_rn(gated_unit<EPI == EPI_GEGLU>(gate, up));
         }
       } else {
 #pragma unroll
@@ -495,7 +496,7 @@ stream_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_const
       // The sums run in member order over this block's own inbox.
       const int tid = threadIdx.x - 64;
       const int plane = p.M * slice;
-      if (EPI == EPI_SWIGLU) {
+      if (gated(EPI)) {
         const int pairs = rows / 2;
         for (int item = tid; item < pairs * p.M; item += 128) {
           const int m = item / pairs, j = item - m * pairs;
@@ -513,7 +514,7 @@ stream_gemm_kernel(const __grid_constant__ CUtensorMap w_map, const __grid_const
           const int n = n0 + r_begin + 2 * j;
           if (n < p.N)
             static_cast<__nv_bfloat16*>(p.y)[static_cast<int64_t>(m) * (p.N / 2) + n / 2] =
-                __float2bfloat16_rn(gate / (1.f + expf(-gate)) * up);
+                __float2bfloat16_rn(gated_unit<EPI == EPI_GEGLU>(gate, up));
         }
       } else {
         for (int item = tid; item < rows * p.M; item += 128) {
@@ -627,14 +628,18 @@ StreamKernel pick_mode(int mode, bool folded, bool traced) {
     default: return pick_form<EPI, MODE_PULL>(folded, traced);
   }
 }
+template <int EPI>
+StreamKernel pick_plain(int mode) {  // epilogues with a plain form only: not around a folded norm (refused), not traced
+  return mode == MODE_SINGLE ? stream_gemm_kernel<EPI, MODE_SINGLE, false, false>
+         : mode == MODE_PUSH ? stream_gemm_kernel<EPI, MODE_PUSH, false, false>
+                             : stream_gemm_kernel<EPI, MODE_PULL, false, false>;
+}
 StreamKernel pick_kernel(int epilogue, int mode, bool folded, bool traced) {
   switch (epilogue) {
     case EPI_F32: return pick_mode<EPI_F32>(mode, folded, traced);
     case EPI_SWIGLU: return pick_mode<EPI_SWIGLU>(mode, folded, traced);
-    case EPI_SQUARED_RELU:  // plain form only: not around a folded norm (refused), not traced
-      return mode == MODE_SINGLE ? stream_gemm_kernel<EPI_SQUARED_RELU, MODE_SINGLE, false, false>
-             : mode == MODE_PUSH ? stream_gemm_kernel<EPI_SQUARED_RELU, MODE_PUSH, false, false>
-                                 : stream_gemm_kernel<EPI_SQUARED_RELU, MODE_PULL, false, false>;
+    case EPI_SQUARED_RELU: return pick_plain<EPI_SQUARED_RELU>(mode);
+    case EPI_GEGLU: return pick_plain<EPI_GEGLU>(mode);
     default: return pick_mode<EPI_BF16>(mode, folded, traced);
   }
 }
@@ -787,10 +792,10 @@ StreamPlan plan_stream(int N, int K, int tokens_pad) {
 constexpr int kStreamMaxRows = 256;
 
 // Shapes the kernel takes: at most 256 rows of X, K a multiple of 8 (row pitch a multiple of 16
-// bytes, which TMA needs), N even for the SwiGLU epilogue.
+// bytes, which TMA needs), N even for the gated epilogues.
 B200_API int b200_stream_gemm_supported(int M, int N, int K, int epilogue) {
   if (M < 1 || M > kStreamMaxRows || N < 1 || K < 8 || K % 8) return 0;
-  if (epilogue == EPI_SWIGLU && N % 2) return 0;
+  if (gated(epilogue) && N % 2) return 0;
   return 1;
 }
 
@@ -854,8 +859,8 @@ B200_API int b200_stream_gemm_fold(const void* W, const void* X, void* Y, int M,
 static int stream_gemm_run(const void* W, const void* X, void* Y, int M, int N, int K, int epilogue, int* err,
                            const NormFold& fold, cudaStream_t stream) {
   B200_REQUIRE(b200_stream_gemm_supported(M, N, K, epilogue), "stream_gemm: unsupported shape %d x %d x %d", M, N, K);
-  B200_REQUIRE(epilogue >= EPI_BF16 && epilogue <= EPI_SQUARED_RELU, "stream_gemm: unknown epilogue %d", epilogue);
-  B200_REQUIRE(epilogue != EPI_SQUARED_RELU || (fold.ss_in == nullptr && fold.x == nullptr), "stream_gemm: the squared relu has no folded form");
+  B200_REQUIRE(epilogue >= EPI_BF16 && epilogue <= EPI_GEGLU, "stream_gemm: unknown epilogue %d", epilogue);
+  B200_REQUIRE(epilogue < EPI_SQUARED_RELU || (fold.ss_in == nullptr && fold.x == nullptr), "stream_gemm: the squared relu and gelu epilogues have no folded form");
   B200_REQUIRE(reinterpret_cast<uintptr_t>(W) % 16 == 0 && reinterpret_cast<uintptr_t>(X) % 16 == 0,
                "stream_gemm: operands must be 16-byte aligned");
   StreamParams p;

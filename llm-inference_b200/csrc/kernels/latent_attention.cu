@@ -8,7 +8,11 @@
 // products around them are matrix products of their own. The softmax's denominator also holds
 // exp(sink[h]), a term without key or value; the head's output is multiplied by
 // sigmoid(gate[t, h]). Scores, weights and sums are 32-bit.
-#include "common.cuh"
+//
+// `latent_kv_write` norms and rotates and writes the rows. Without a rotated part (rot_dim 0) nothing of a row depends on the
+// token's position, and `latent_norms_write` takes its place: the norm of the latent with its page write and, where the
+// queries come out of a latent of their own, that one's norm, in one kernel in front of the queries' product.
+#include "packs.cuh"
 
 namespace {
 
@@ -88,6 +92,45 @@ __global__ void latent_kv_write_kernel(const T* q_proj, int q_ld, const T* proj,
       dst[rank + rot_dims + i - half] = kv[rank + rot_dims + i - half];
     }
   }
+}
+
+// One block per token: [q latent (q_rank, may be 0)] at q_at and [latent (rank)] at kv_at of the token's row of `proj`, each over
+// its root mean square times its weight, to q_out [tokens][q_rank] and to the token's cache row of `rank` numbers. W numbers an access.
+template <typename T, int W>
+__global__ void latent_norms_write_kernel(const T* proj, int ld, int q_at, int q_rank, const float* __restrict__ q_weight, T* q_out,
+                                          int kv_at, int rank, const float* __restrict__ norm_weight, float eps, const int* __restrict__ positions,
+                                          const int* __restrict__ token_seq, const int* __restrict__ block_table, int max_pages, int num_pages,
+                                          T* arena, int page_size, int writes, int* err) {
+  __shared__ float scratch[32];
+  let_successor_start();
+  const int t = blockIdx.x, tid = threadIdx.x;
+  const int pos = positions[t];
+  int page = -1;
+  if (writes) {
+    const int logical = pos / page_size;
+    page = (pos >= 0 && logical < max_pages) ? block_table[static_cast<int64_t>(token_seq[t]) * max_pages + logical] : -1;
+    if (page < 0 || page >= num_pages) {
+      if (tid == 0) atomicOr(err, pos >= 0 && logical < max_pages ? ERRBIT_BAD_PAGE : ERRBIT_BAD_POSITION);
+      page = -1;
+    }
+  }
+  wait_for_predecessor();
+  const T* row = proj + static_cast<int64_t>(t) * ld;
+  float ss_q = 0.f, ss_kv = 0.f;
+  for (int i = tid * W; i < q_rank; i += blockDim.x * W) ss_q = square_sum(Pack<W>::load(row + q_at + i), ss_q);
+  for (int i = tid * W; i < rank; i += blockDim.x * W) ss_kv = square_sum(Pack<W>::load(row + kv_at + i), ss_kv);
+  if (q_rank > 0) {
+    const float inv = 1.f / sqrtf(block_sum(ss_q, scratch) / static_cast<float>(q_rank) + eps);
+    T* dst = q_out + static_cast<int64_t>(t) * q_rank;
+    for (int i = tid * W; i < q_rank; i += blockDim.x * W)
+      Pack<W>::store(dst + i, mul_each(scale_each(Pack<W>::load(row + q_at + i), inv), Pack<W>::load(q_weight + i)));
+  }
+  if (!writes) return;
+  const float inv = 1.f / sqrtf(block_sum(ss_kv, scratch) / static_cast<float>(rank) + eps);
+  if (page < 0) return;
+  T* dst = arena + (static_cast<int64_t>(page) * page_size + pos % page_size) * rank;
+  for (int i = tid * W; i < rank; i += blockDim.x * W)
+    Pack<W>::store(dst + i, mul_each(scale_each(Pack<W>::load(row + kv_at + i), inv), Pack<W>::load(norm_weight + i)));
 }
 
 template <typename T>
@@ -207,6 +250,36 @@ B200_API int b200_latent_kv_write(const void* q_proj, int q_ld, const void* proj
     return b200_fail("latent_kv_write: unknown dtype %d", dtype);
   }
   return b200_check_launch("latent_kv_write");
+}
+
+// `writes` 0 leaves the cache alone; `q_rank` 0: the queries have no latent of their own.
+B200_API int b200_latent_norms_write(const void* proj, int ld, int q_at, int q_rank, const float* q_weight, void* q_out, int kv_at, int rank,
+                                     const float* norm_weight, float eps, const int* positions, const int* token_seq, const int* block_table,
+                                     int max_pages, int num_pages, void* arena, int page_size, int tokens, int writes, int dtype, int* err,
+                                     cudaStream_t stream) {
+  if (tokens == 0) return 0;
+  B200_REQUIRE(tokens > 0 && rank > 0 && q_rank >= 0 && q_at >= 0 && kv_at >= 0 && q_at + q_rank <= ld && kv_at + rank <= ld,
+               "latent_norms_write: rows of %d numbers do not hold the latents", ld);
+  B200_REQUIRE(q_rank == 0 || (q_weight != nullptr && q_out != nullptr), "latent_norms_write: the queries' latent has no weight or output");
+  B200_REQUIRE(page_size > 0 && max_pages > 0, "latent_norms_write: bad geometry");
+  const bool wide = (q_rank == 0 || packs_of_four(q_rank, q_weight, q_out)) && packs_of_four(rank, proj, norm_weight, arena) && ld % 4 == 0 &&
+                    q_at % 4 == 0 && kv_at % 4 == 0;
+  const int threads = max(rank, q_rank) > (wide ? 512 : 128) ? 256 : 128;
+  auto launch = [&](auto kernel, auto zero) {
+    using T = decltype(zero);
+    launch_kernel(kernel, dim3(tokens), dim3(threads), 0, stream, static_cast<const T*>(proj), ld, q_at, q_rank, q_weight, static_cast<T*>(q_out), kv_at,
+                  rank, norm_weight, eps, positions, token_seq, block_table, max_pages, num_pages, static_cast<T*>(arena), page_size, writes, err);
+  };
+  if (dtype == DTYPE_F32) {
+    if (wide) launch(latent_norms_write_kernel<float, 4>, float{});
+    else launch(latent_norms_write_kernel<float, 1>, float{});
+  } else if (dtype == DTYPE_BF16) {
+    if (wide) launch(latent_norms_write_kernel<__nv_bfloat16, 4>, __nv_bfloat16{});
+    else launch(latent_norms_write_kernel<__nv_bfloat16, 1>, __nv_bfloat16{});
+  } else {
+    return b200_fail("latent_norms_write: unknown dtype %d", dtype);
+  }
+  return b200_check_launch("latent_norms_write");
 }
 
 B200_API int b200_latent_attention_plain(const void* q_lat, int64_t q_lat_token, int64_t q_lat_head, const void* q_rot,

@@ -51,17 +51,18 @@ _SIGNATURES: dict[str, list] = {
     "b200_embedding_gather": [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_int, c_void_p, c_void_p],
     "b200_rmsnorm": [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_float, c_int, c_void_p],
     "b200_silu_mul": [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
+    "b200_gelu_mul": [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p],
     "b200_rope_kv_write": [c_void_p] * 7 + [c_int, c_int] + [c_void_p] * 3 + [c_int] * 8 + [c_void_p, c_void_p],
     "b200_paged_attention_plain": [c_void_p] * 6
     + [c_int, c_int, c_void_p]
     + [c_int] * 7
-    + [c_float, c_int, c_float, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p],
+    + [c_float, c_int, c_float, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p, c_void_p],
     "b200_gemm_f32": [c_void_p] * 4 + [c_int] * 6 + [c_void_p],
     "b200_paged_flash_attention": [c_void_p] * 8 + [c_int] * 12 + [c_float, c_int, c_int, c_int, c_float, c_void_p, c_int, c_int, c_void_p,
-                                   c_void_p, c_void_p, c_void_p],
-    "b200_paged_decode_attention_tma": [c_void_p] * 8 + [c_int] * 9 + [c_float, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p],
+                                   c_void_p, c_void_p, c_void_p, c_void_p],
+    "b200_paged_decode_attention_tma": [c_void_p] * 8 + [c_int] * 9 + [c_float, c_int, c_int] + [c_void_p] * 5,
     "b200_flash_prefill_tcgen05": [c_void_p] * 8 + [c_int] * 12 + [c_float, c_int, c_float, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p,
-                                   c_void_p],
+                                   c_void_p, c_void_p],
     "b200_skinny_gemm": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int64, c_void_p, c_int, c_void_p],
     "b200_stream_gemm": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
     "b200_skinny_gemm_fold": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_int64, c_void_p, c_int,
@@ -78,15 +79,20 @@ _SIGNATURES: dict[str, list] = {
     "b200_poly_norm": [c_void_p, c_void_p, c_int, c_int, c_float, c_void_p, c_int, c_void_p],
     "b200_latent_kv_write": [c_void_p, c_int, c_void_p] + [c_int] * 8 + [c_void_p, c_float, c_void_p, c_int, c_int, c_float] + [c_void_p] * 3
                             + [c_int, c_int, c_void_p, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p],
+    "b200_latent_norms_write": [c_void_p, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_float] + [c_void_p] * 3
+                               + [c_int, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
     "b200_latent_attention_plain": [c_void_p, c_int64, c_int64] + [c_void_p] * 5 + [c_int, c_int, c_void_p, c_void_p, c_int64,
                                     c_void_p, c_int64, c_int64] + [c_int] * 6 + [c_float, c_int, c_void_p, c_void_p],
     "b200_latent_attention_mma": [c_void_p, c_int64, c_int64, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int] + [c_void_p] * 3
                                  + [c_int, c_int, c_int, c_void_p, c_void_p, c_int64, c_void_p, c_int64, c_int64, c_int, c_int, c_int,
                                     c_float, c_int, c_void_p, c_void_p, c_void_p],
-    "b200_delta_prepare": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int] + [c_void_p] * 7 + [c_int] * 6 + [c_void_p] * 5
+    "b200_delta_prepare": [c_void_p, c_int, c_void_p, c_int, c_void_p, c_int] + [c_void_p] * 7 + [c_int] * 6 + [c_void_p] * 6
                           + [c_int, c_void_p],
     "b200_delta_recurrence": [c_void_p] * 8 + [c_int] * 5 + [c_void_p] * 3,
-    "b200_delta_output": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_void_p, c_int, c_void_p],
+    "b200_delta_output": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_int, c_void_p],
+    "b200_delta_head_recurrence": [c_void_p] * 9 + [c_int] * 6 + [c_void_p] * 3,
+    "b200_delta_head_step": [c_void_p, c_int, c_void_p, c_int] + [c_void_p] * 4 + [c_float, c_void_p, c_void_p] + [c_int] * 5
+                            + [c_void_p, c_void_p, c_int, c_void_p],
     "b200_embedding_sinusoid": [c_void_p] * 4 + [c_float, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
     "b200_hyper_norm": [c_void_p] * 7 + [c_int, c_int, c_int, c_float, c_void_p, c_int, c_void_p],
     "b200_softcap": [c_void_p, c_int64, c_float, c_void_p],
@@ -159,6 +165,8 @@ class KernelLibrary:
         self.lib.b200_latent_attention_mma_supported.restype = c_int
         self.lib.b200_latent_attention_mma_scratch.argtypes = [c_int] * 5
         self.lib.b200_latent_attention_mma_scratch.restype = c_int64
+        self.lib.b200_delta_head_step_supported.argtypes = [c_int] * 4
+        self.lib.b200_delta_head_step_supported.restype = c_int
         self.lib.b200_moe_tile_rows.argtypes = []
         self.lib.b200_moe_tile_rows.restype = c_int
         self.lib.b200_moe_mma_supported.argtypes = [c_int, c_int]

@@ -1,4 +1,4 @@
-"""A recurrent mixer: the gated delta rule with a decay per head and key channel."""
+"""Recurrent mixers: the gated delta rule with a decay per head and key channel or one per head, and its generalized form."""
 
 from __future__ import annotations
 
@@ -105,6 +105,80 @@ class ChannelDeltaRule(Part):
         return ops.linear(ctx, y, self.w_o, ctx.buffer("branch", (t, self.hidden_size)))
 
 
+class HeadDeltaRule(Part):
+    """The gated delta rule with one decay per head: ``S = g S``; ``u = beta (v - S^T k)``; ``S = S + k u^T``; ``o = S^T q`` over a
+    state ``S [dim, vdim]`` per head (32-bit, zero at a request's start).
+
+    ``q, k`` (``kv_heads x dim``, head ``n`` uses q/k head ``n // (heads / kv_heads)``), ``v`` (``heads x vdim``), their short
+    convolutions with silu, unit vectors and ``beta`` are those of :class:`ChannelDeltaRule`.
+    ``g = exp(-exp(A_log[n]) * softplus((W_a h)[n] + dt_bias[n]))``. Each head's ``o`` is divided by its root mean square over
+    ``vdim``, times ``norm`` (shared by the heads), times ``silu(W_g h)`` (``heads x vdim``); then ``W_o``.
+
+    All projections of ``h`` are one matrix ``[q | k | v | b | a | g]``. A step of single tokens runs everything between the two
+    products as one kernel. Per-request state: ``S`` and the convolution's last ``taps - 1`` inputs. Tensor names are
+    ``prefix + q | q.conv | k | k.conv | v | v.conv | b | A_log | norm | a | dt_bias | g | o``."""
+
+    def __init__(self, *, prefix: str, hidden_size: int, heads: int, kv_heads: int, dim: int, vdim: int, taps: int, eps: float,
+                 out_name: str = "branch") -> None:
+        if heads % kv_heads:
+            raise ValueError(f"{heads} heads cannot share {kv_heads} q/k heads")
+        if taps < 1:
+            raise ValueError("the convolution needs at least the current token's tap")
+        self.prefix, self.hidden_size, self.out_name = prefix, hidden_size, out_name
+        self.heads, self.kv_heads, self.dim, self.vdim, self.taps, self.eps = heads, kv_heads, dim, vdim, int(taps), float(eps)
+        self.channels = 2 * kv_heads * dim + heads * vdim
+        self.dtype = torch.bfloat16
+        self.w_in = self.w_o = self.taps_w = self.a_log = self.dt_bias = self.norm_weight = None
+
+    def cache_spec(self) -> StateSpec:
+        return StateSpec(((self.heads, self.dim, self.vdim), (self.taps - 1, self.channels)), (torch.float32, self.dtype))
+
+    def tensor_specs(self) -> list[TensorSpec]:
+        p, d = self.prefix, self.hidden_size
+        qk, vw = self.kv_heads * self.dim, self.heads * self.vdim
+        specs = []
+        for name, width in (("q", qk), ("k", qk), ("v", vw)):
+            specs += [TensorSpec(p + name, (width, d)), TensorSpec(p + name + ".conv", (width, self.taps), init="half_plus_normal")]
+        return specs + [
+            TensorSpec(p + "b", (self.heads, d)), TensorSpec(p + "a", (self.heads, d)), TensorSpec(p + "A_log", (self.heads,)),
+            TensorSpec(p + "dt_bias", (self.heads,)), TensorSpec(p + "norm", (self.vdim,), init="one_plus_normal"),
+            TensorSpec(p + "g", (vw, d)), TensorSpec(p + "o", (d, vw)),
+        ]
+
+    def load(self, tensors, dtype, device) -> None:
+        p, f32 = self.prefix, torch.float32
+        self.dtype = dtype
+
+        def get(name: str, to=dtype) -> torch.Tensor:
+            return tensors[p + name].to(device=device, dtype=to).contiguous()
+
+        self.w_in = torch.cat([get(n) for n in ("q", "k", "v", "b", "a", "g")]).contiguous()
+        self.w_o = get("o")
+        self.taps_w = torch.cat([get(n + ".conv", f32) for n in ("q", "k", "v")]).contiguous()
+        self.a_log, self.dt_bias, self.norm_weight = get("A_log", f32), get("dt_bias", f32), get("norm", f32)
+
+    def weight_bytes(self) -> int:
+        return sum(w.numel() * w.element_size() for w in (self.w_in, self.w_o))
+
+    def forward(self, ctx: StepContext, cache: CacheView, h: torch.Tensor) -> torch.Tensor:
+        t, heads, kvh, dk, dv = ctx.num_tokens, self.heads, self.kv_heads, self.dim, self.vdim
+        state, conv_state = cache.state
+        proj = ops.linear(ctx, h, self.w_in, ctx.buffer("delta_in", (t, self.w_in.shape[0])))
+        y = ctx.buffer("attn", (t, heads * dv))
+        if ops.delta_head_step_takes(ctx, heads, kvh, dk, dv):
+            ops.delta_head_step(ctx, proj, self.taps_w, conv_state, self.a_log, self.dt_bias, self.norm_weight, self.eps, state, y, heads, kvh, dk, dv)
+        else:
+            f32 = torch.float32
+            widths = (("q", kvh * dk), ("k", kvh * dk), ("v", heads * dv), ("beta", heads), ("decay", heads), ("kq", kvh))
+            q, k, v, beta, decay, kq = (ctx.buffer("delta_" + name, (t, width), f32) for name, width in widths)
+            a_at = self.channels + heads
+            ops.delta_prepare(ctx, proj, proj[:, a_at : a_at + heads], self.taps_w, conv_state, self.a_log, self.dt_bias, heads, kvh, dk, dv,
+                              q, k, v, beta, decay, kq)
+            o = ops.delta_head_recurrence(ctx, q, k, v, beta, decay, kq, state, ctx.buffer("delta_o", (t, heads * dv), f32), heads, kvh, dk, dv)
+            ops.delta_output(ctx, o, self.norm_weight, proj[:, a_at + heads :], heads, dv, self.eps, y, silu=True)
+        return ops.linear(ctx, y, self.w_o, ctx.buffer(self.out_name, (t, self.hidden_size)))
+
+
 class GeneralDeltaRule(Part):
     """Per head a state ``S [dim, dim]`` (32-bit, zero at a request's start) is carried from token to token:
     ``S <- diag(w) S - (a * u) (u^T S) + k v^T`` (both terms read the old state), ``o = S^T r`` (the new one), with
@@ -167,4 +241,5 @@ class GeneralDeltaRule(Part):
 
 
 register_part("mixer", "channel_delta", ChannelDeltaRule)
+register_part("mixer", "head_delta", HeadDeltaRule)
 register_part("mixer", "general_delta", GeneralDeltaRule)

@@ -16,6 +16,9 @@ class SwiGLU(Part):
     rows interleaved (row 2j is gate_j, row 2j + 1 is up_j), so one matrix product yields each
     gate next to its up value and the activation can run in that product's epilogue."""
 
+    activation = "silu"
+    names = ("gate_proj.weight", "up_proj.weight", "down_proj.weight")
+
     def __init__(self, *, prefix: str, hidden_size: int, intermediate_size: int) -> None:
         self.prefix, self.hidden_size, self.intermediate_size = prefix, hidden_size, intermediate_size
         self.w_gate_up = self.w_down = None
@@ -23,16 +26,16 @@ class SwiGLU(Part):
     def tensor_specs(self) -> list[TensorSpec]:
         p, h, i = self.prefix, self.hidden_size, self.intermediate_size
         return [
-            TensorSpec(f"{p}gate_proj.weight", (i, h)),
-            TensorSpec(f"{p}up_proj.weight", (i, h)),
-            TensorSpec(f"{p}down_proj.weight", (h, i)),
+            TensorSpec(p + self.names[0], (i, h)),
+            TensorSpec(p + self.names[1], (i, h)),
+            TensorSpec(p + self.names[2], (h, i)),
         ]
 
     def load(self, tensors, dtype, device) -> None:
         p = self.prefix
-        gate, up = (tensors[f"{p}{n}.weight"].to(device=device, dtype=dtype) for n in ("gate_proj", "up_proj"))
+        gate, up = (tensors[p + n].to(device=device, dtype=dtype) for n in self.names[:2])
         self.w_gate_up = torch.stack([gate, up], dim=1).reshape(2 * self.intermediate_size, self.hidden_size).contiguous()
-        self.w_down = tensors[f"{p}down_proj.weight"].to(device=device, dtype=dtype).contiguous()
+        self.w_down = tensors[p + self.names[2]].to(device=device, dtype=dtype).contiguous()
 
     def weight_bytes(self) -> int:
         return (self.w_gate_up.numel() + self.w_down.numel()) * self.w_down.element_size()
@@ -43,14 +46,23 @@ class SwiGLU(Part):
     def forward(self, ctx: StepContext, h, sink: ops.ResidualSink | None = None):
         t, i = ctx.num_tokens, self.intermediate_size
         act = ctx.buffer("act", (t, i))
-        if not ops.linear_swiglu(ctx, h, self.w_gate_up, act):
+        if not ops.linear_gated(ctx, h, self.w_gate_up, act, self.activation):
             gate_up = ops.linear(ctx, h, self.w_gate_up, ctx.buffer("gate_up", (t, 2 * i)))
-            ops.silu_mul(ctx, gate_up, act)
+            ops.gated_mul(ctx, gate_up, act, self.activation)
         if sink is not None:
             folded = ops.linear_into_residual(ctx, act, self.w_down, sink)
             if folded is not None:
                 return folded
         return ops.linear(ctx, act, self.w_down, ctx.buffer("branch", (t, self.hidden_size)))
+
+
+class GeGLU(SwiGLU):
+    """``down(gelu(gate(h)) * up(h))`` without biases, ``gelu`` in its tanh form: the same products with another activation
+    in the first one's epilogue (which has no form for a folded norm's rows). Tensor names: ``prefix + gate | up | down``."""
+
+    activation = "gelu"
+    names = ("gate", "up", "down")
+    takes_folded = False
 
 
 class PolyNormFeedForward(Part):
@@ -255,6 +267,7 @@ class SquaredReLUFeedForward(Part):
 
 
 register_part("feed_forward", "swiglu", SwiGLU)
+register_part("feed_forward", "geglu", GeGLU)
 register_part("feed_forward", "poly_norm", PolyNormFeedForward)
 register_part("feed_forward", "routed_experts", RoutedExperts)
 register_part("feed_forward", "clamped_glu", ClampedGLU)

@@ -27,16 +27,20 @@ class LatentAttention(Part):
     With ``q_rank`` the queries come out of a latent of their own: ``q = W_uq rmsnorm(W_dq h)`` (weight ``dq.norm``)
     instead of ``W_q h``. With ``gate_per="element"`` the gate is one number per output number: the concatenated heads are
     multiplied element by element by ``sigmoid(W_g h)`` (``W_g`` is ``[heads * vdim, hidden]``) after the expansion by
-    ``W_uv``. The position part may pair neighbours or halves of the rotated part.
+    ``W_uv``. The position part may pair neighbours or halves of the rotated part. Without a rotated part (``rot_dim`` 0,
+    ``position`` None) positions do not enter at all: the cached row is the latent alone, and both latents' norms and the
+    cache write are one kernel.
 
     The query (or its latent), latent and gate projections are one matrix product. Tensor names are
     ``prefix + q | dq | dq.norm | uq | dkv | dkv.norm | uk | uv | sink | g | o``."""
 
     def __init__(self, *, prefix: str, hidden_size: int, heads: int, dim: int, rot_dim: int, vdim: int, rank: int,
-                 scale: float, eps: float, position: PartSpec, sink: bool = True, gate: bool = True, window: int = 0,
+                 scale: float, eps: float, position: PartSpec | None = None, sink: bool = True, gate: bool = True, window: int = 0,
                  q_rank: int | None = None, gate_per: str = "head", out_name: str = "branch") -> None:
         if gate_per not in ("head", "element"):
             raise ValueError(f"gate_per={gate_per!r} must be 'head' or 'element'")
+        if (position is None) != (rot_dim == 0):
+            raise ValueError("a rotated part and a position encoding come together")
         self.prefix, self.hidden_size, self.out_name = prefix, hidden_size, out_name
         self.q_rank = int(q_rank) if q_rank else 0
         self.gate_per_element = bool(gate) and gate_per == "element"
@@ -44,8 +48,8 @@ class LatentAttention(Part):
         self.heads, self.dim, self.rot_dim, self.vdim, self.rank = heads, dim, rot_dim, vdim, rank
         self.scale, self.eps, self.window = float(scale), float(eps), int(window)
         self.has_sink, self.has_gate = bool(sink), bool(gate)
-        self.position = build_part("position", position)
-        self.graph_safe = self.position.graph_safe
+        self.position = build_part("position", position) if position is not None else None
+        self.graph_safe = self.position.graph_safe if self.position is not None else True
         self.w_in = self.w_uk_t = self.w_uv = self.w_o = self.sink = self.norm_weight = None
 
     def cache_spec(self) -> KVCacheSpec:
@@ -70,7 +74,7 @@ class LatentAttention(Part):
             specs.append(TensorSpec(p + "sink", (self.heads,)))
         if self.has_gate:
             specs.append(TensorSpec(p + "g", (self.heads * self.vdim if self.gate_per_element else self.heads, d)))
-        return specs + self.position.tensor_specs()
+        return specs + (self.position.tensor_specs() if self.position is not None else [])
 
     def load(self, tensors, dtype, device) -> None:
         p = self.prefix
@@ -85,7 +89,8 @@ class LatentAttention(Part):
         self.w_o = tensors[p + "o"].to(device=device, dtype=dtype).contiguous()
         self.norm_weight = tensors[p + "dkv.norm"].to(device=device, dtype=torch.float32).contiguous()
         self.sink = tensors[p + "sink"].to(device=device, dtype=torch.float32).contiguous() if self.has_sink else None
-        self.position.load(tensors, dtype, device)
+        if self.position is not None:
+            self.position.load(tensors, dtype, device)
 
     def weight_bytes(self) -> int:
         return sum(w.numel() * w.element_size() for w in (self.w_in, self.w_uk_t, self.w_uv, self.w_o, self.w_uq) if w is not None)
@@ -96,7 +101,13 @@ class LatentAttention(Part):
         width = self.w_in.shape[0]
         proj = ops.linear(ctx, h, self.w_in, ctx.buffer("latent_in", (t, width)))
         q_rot = ctx.buffer("latent_q_rot", (t, heads * rot))
-        if self.q_rank:
+        if self.position is None:
+            # nothing depends on the position: both latents' norms and the cache write are one kernel in front of the queries
+            latent_q = ctx.buffer("latent_cq", (t, self.q_rank)) if self.q_rank else None
+            kv_offset = self.q_rank or q_width
+            ops.latent_norms_write(ctx, cache, proj, 0, kv_offset, rank, self.norm_weight, self.eps, self.q_norm_weight, latent_q)
+            queries = ops.linear(ctx, latent_q, self.w_uq, ctx.buffer("latent_queries", (t, q_width))) if self.q_rank else proj[:, :q_width]
+        elif self.q_rank:
             # queries through their own latent: norm of the first q_rank columns, then one more product
             latent_q = ops.rms_rows(ctx, proj[:, : self.q_rank], self.q_norm_weight, self.eps, ctx.buffer("latent_cq", (t, self.q_rank)))
             queries = ops.linear(ctx, latent_q, self.w_uq, ctx.buffer("latent_queries", (t, q_width)))

@@ -188,9 +188,14 @@ def _choose_small_gemm(ctx: StepContext, m: int, n: int, k: int, epilogue: int, 
     return "stream" if stream else ("skinny" if skinny else None)
 
 
-def linear_swiglu(ctx: StepContext, x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor) -> bool:
+GATED_EPILOGUES = {"silu": 2, "gelu": 4}  # of this engine's own products, over interleaved gate/up rows
+
+
+def linear_gated(ctx: StepContext, x: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, activation: str = "silu") -> bool:
     """``out = silu(gate) * up`` of ``x @ weight.T`` with interleaved gate/up rows, in one
-    kernel. Returns False (doing nothing) when no fused kernel takes the shape."""
+    kernel; ``activation="gelu"``: the tanh form of gelu instead of silu (not on a folded norm's rows).
+    Returns False (doing nothing) when no fused kernel takes the shape."""
+    epilogue = GATED_EPILOGUES[activation]
     folded = x if isinstance(x, FoldedRows) else None
     if folded is not None:
         x = folded.xn
@@ -198,11 +203,11 @@ def linear_swiglu(ctx: StepContext, x: torch.Tensor, weight: torch.Tensor, out: 
     n = weight.shape[0]
     if x.dtype != torch.bfloat16 or m == 0:
         return False
-    kernel = _small_gemm_kernel(ctx, m, n, k, 2)
-    if kernel is None or (folded is not None and not fold_enabled(ctx)):
+    kernel = _small_gemm_kernel(ctx, m, n, k, epilogue)
+    if kernel is None or (folded is not None and (activation != "silu" or not fold_enabled(ctx))):
         return False
-    _need(tuple(out.shape) == (m, n // 2) and out.is_contiguous() and x.is_contiguous(), "linear_swiglu: bad operands")
-    _small_gemm(ctx, kernel, x, weight, out, 2, scale=folded)
+    _need(tuple(out.shape) == (m, n // 2) and out.is_contiguous() and x.is_contiguous(), "linear_gated: bad operands")
+    _small_gemm(ctx, kernel, x, weight, out, epilogue, scale=folded)
     return True
 
 
@@ -308,13 +313,14 @@ def rmsnorm(
     return out
 
 
-def silu_mul(ctx: StepContext, gate_up: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+def gated_mul(ctx: StepContext, gate_up: torch.Tensor, out: torch.Tensor, activation: str = "silu") -> torch.Tensor:
+    """``out = silu(gate) * up`` (or gelu, its tanh form) of interleaved gate/up columns."""
     tokens, twice = gate_up.shape
     inter = twice // 2
-    _need(twice == 2 * inter and tuple(out.shape) == (tokens, inter), "silu_mul: bad shapes")
-    _need(gate_up.is_contiguous() and out.is_contiguous() and gate_up.dtype == out.dtype, "silu_mul: bad operands")
+    _need(twice == 2 * inter and tuple(out.shape) == (tokens, inter), "gated_mul: bad shapes")
+    _need(gate_up.is_contiguous() and out.is_contiguous() and gate_up.dtype == out.dtype, "gated_mul: bad operands")
     ctx.lib.call(
-        "b200_silu_mul", ptr(gate_up), ptr(out), c_int(tokens), c_int(inter), c_int(dtype_code(out.dtype)), ctx.stream,
+        f"b200_{activation}_mul", ptr(gate_up), ptr(out), c_int(tokens), c_int(inter), c_int(dtype_code(out.dtype)), ctx.stream,
     )
     return out
 
@@ -353,16 +359,17 @@ class ScoreShape:
     (``s <- softcap * tanh(s / softcap)``), ``bias`` (float32 ``[q_heads, reach + 1]`` on the device: the row of the
     query head at ``min(position - key, reach)`` is added after the cap) and ``chunk`` (a query sees only keys from
     ``floor(position / chunk) * chunk`` on). The plain kernel, the ``mma.sync`` kernels and the tcgen05 prefill
-    kernel take it (the last wants ``bias_peak`` beside a bias)."""
+    kernel take it (the last wants ``bias_peak`` beside a bias). ``sink`` goes with every softmax form of every kernel."""
 
     softcap: float = 0.0
     bias: torch.Tensor | None = None
     chunk: int = 0
     bias_peak: torch.Tensor | None = None  # float32 [q_heads]: each row's largest entry (the tcgen05 kernel bounds exponents with it)
     sigmoid_bias: torch.Tensor | None = None  # float32 [q_heads]: a visible key weighs sigmoid(score + bias), nothing is normalised
+    sink: torch.Tensor | None = None  # float32 [q_heads]: the softmax's denominator also holds exp(sink), without key or value, not scaled
 
     def __bool__(self) -> bool:
-        return self.changes_scores() or self.sigmoid_bias is not None
+        return self.changes_scores() or self.sigmoid_bias is not None or self.sink is not None
 
     def changes_scores(self) -> bool:
         """Whether a score is more than the scaled product (the TMA decode kernel takes none of that)."""
@@ -379,8 +386,10 @@ class ScoreShape:
                   "attention: the bias by distance is float32 [q_heads, reach + 1]")
         if self.sigmoid_bias is not None:
             _need(self.sigmoid_bias.dtype == torch.float32 and self.sigmoid_bias.numel() == q_heads, "attention: the sigmoid's bias is float32 [q_heads]")
+        _need(self.sink is None or (self.sink.dtype == torch.float32 and self.sink.numel() == q_heads), "attention: the sink is float32 [q_heads]")
+        _need(self.sink is None or self.sigmoid_bias is None, "attention: a sink is a term of a softmax, sigmoid weights have none")
         reach = self.bias.shape[1] - 1 if self.bias is not None else 0
-        return [c_float(self.softcap), ptr(self.bias), c_int(reach), c_int(self.chunk), ptr(self.sigmoid_bias)]
+        return [c_float(self.softcap), ptr(self.bias), c_int(reach), c_int(self.chunk), ptr(self.sigmoid_bias), ptr(self.sink)]
 
 
 NO_SHAPE = ScoreShape()
@@ -538,7 +547,7 @@ def paged_flash_attention(
             ptr(ctx.seq_q_start), ptr(ctx.seq_q_len), ptr(ctx.seq_kv_len), c_int(num_seqs), c_int(cache.max_pages),
             c_int(cache.num_pages), c_int(q_heads), c_int(kv_heads), c_int(head_dim), c_int(cache.page_size),
             c_int(cache.window), c_int(cache.keep_first), c_float(scale), c_int(splits), c_int(int(ctx.options.get("decode_stages", DECODE_STAGES))),
-            ptr(shape.sigmoid_bias), ptr(scratch), ptr(ctx.err), ctx.stream,
+            *shape.arguments(q_heads)[4:], ptr(scratch), ptr(ctx.err), ctx.stream,
         )
         if scratch is not None:
             ctx.lib.calls += 1  # the merge kernel is a launch of its own
@@ -590,7 +599,7 @@ def paged_prefill_attention_tcgen05(
         ptr(ctx.seq_q_start), ptr(ctx.seq_q_len), ptr(ctx.seq_kv_len), c_int(first_seq), c_int(num_seqs), c_int(max_q_len),
         c_int(ctx.max_kv_len), c_int(cache.max_pages), c_int(cache.num_pages), c_int(q_heads), c_int(kv_heads),
         c_int(head_dim), c_int(cache.page_size), c_int(cache.window), c_int(cache.keep_first), c_float(scale), c_int(value_head), c_float(shape.softcap),
-        ptr(shape.bias), ptr(shape.bias_peak), reach, c_int(shape.chunk), ptr(shape.sigmoid_bias), ptr(ctx.err), ctx.stream,
+        ptr(shape.bias), ptr(shape.bias_peak), reach, c_int(shape.chunk), ptr(shape.sigmoid_bias), ptr(shape.sink), ptr(ctx.err), ctx.stream,
     )
     return out
 
@@ -743,6 +752,26 @@ def latent_kv_write(
     )
 
 
+def latent_norms_write(ctx: StepContext, cache: CacheView, proj: torch.Tensor, q_at: int, kv_at: int, rank: int, norm_weight: torch.Tensor, eps: float,
+                       q_weight: torch.Tensor | None = None, q_out: torch.Tensor | None = None) -> None:
+    """For a latent cache without a rotated part: the ``rank`` numbers from column ``kv_at`` of a token's row of ``proj`` over
+    their root mean square times ``norm_weight`` go to the token's cache row; with ``q_out`` its columns' worth of numbers
+    from ``q_at`` likewise, with ``q_weight``, to ``q_out`` (the queries' own latent)."""
+    tokens, ld = proj.shape
+    q_rank = q_out.shape[1] if q_out is not None else 0
+    _need(proj.is_contiguous() and cache.keys.dtype == proj.dtype, "latent_norms_write: bad operands")
+    _need(norm_weight.dtype == torch.float32 and norm_weight.numel() == rank, "latent_norms_write: the latent's weight is float32 [rank]")
+    _need(tuple(cache.keys.shape[1:]) == (1, cache.page_size, rank), "latent_norms_write: the cache rows are the latents")
+    if q_out is not None:
+        _need(q_out.dtype == proj.dtype and q_out.shape[0] == tokens and q_out.is_contiguous(), "latent_norms_write: bad query latent")
+        _need(q_weight is not None and q_weight.dtype == torch.float32 and q_weight.numel() == q_rank, "latent_norms_write: the query latent's weight is float32 [q_rank]")
+    ctx.lib.call(
+        "b200_latent_norms_write", ptr(proj), c_int(ld), c_int(q_at), c_int(q_rank), ptr(q_weight), ptr(q_out), c_int(kv_at), c_int(rank), ptr(norm_weight),
+        c_float(eps), ptr(ctx.positions), ptr(ctx.token_seq), ptr(cache.block_table), c_int(cache.max_pages), c_int(cache.num_pages), ptr(cache.keys),
+        c_int(cache.page_size), c_int(tokens), c_int(1 if cache.writes else 0), c_int(dtype_code(proj.dtype)), ptr(ctx.err), ctx.stream,
+    )
+
+
 def latent_attention_plain(
     ctx: StepContext, cache: CacheView, q_lat: torch.Tensor, q_rot: torch.Tensor, sink: torch.Tensor | None,
     gate: torch.Tensor | None, out: torch.Tensor, heads: int, rank: int, rot_dim: int, scale: float,
@@ -816,23 +845,26 @@ def latent_attention_mma(
 def delta_prepare(
     ctx: StepContext, proj: torch.Tensor, decay_in: torch.Tensor, taps: torch.Tensor, conv_state: torch.Tensor, a_log: torch.Tensor,
     dt_bias: torch.Tensor, heads: int, kv_heads: int, dk: int, dv: int, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor,
-    beta: torch.Tensor, decay: torch.Tensor,
+    beta: torch.Tensor, decay: torch.Tensor, kq: torch.Tensor | None = None,
 ) -> None:
     """Convolution + silu of the q, k, v columns of ``proj`` (continuing each request's slot of
-    ``conv_state``, which is then moved on), unit vectors, beta and the decay factors, all 32-bit."""
+    ``conv_state``, which is then moved on), unit vectors, beta and the decay factors, all 32-bit.
+    With ``kq`` (``[tokens, kv_heads]``, takes k . q) there is one decay per head and ``decay`` takes its logarithm."""
+    span = dk if kq is None else 1
     tokens = proj.shape[0]
     channels = 2 * kv_heads * dk + heads * dv
     _need(proj.stride(1) == 1 and proj.shape[1] >= channels + heads, "delta_prepare: bad projections")
-    _need(decay_in.stride(1) == 1 and decay_in.shape[1] >= heads * dk and decay_in.dtype == proj.dtype, "delta_prepare: bad decay input")
+    _need(decay_in.stride(1) == 1 and decay_in.shape[1] >= heads * span and decay_in.dtype == proj.dtype, "delta_prepare: bad decay input")
     _need(taps.dtype == torch.float32 and taps.shape[0] == channels and taps.is_contiguous(), "delta_prepare: taps are float32 [channels, taps]")
     _need(conv_state.dtype == proj.dtype and tuple(conv_state.shape[1:]) == (max(taps.shape[1] - 1, 0), channels), "delta_prepare: bad convolution state")
-    for tensor, width in ((q, kv_heads * dk), (k, kv_heads * dk), (v, heads * dv), (beta, heads), (decay, heads * dk)):
+    outputs = [(q, kv_heads * dk), (k, kv_heads * dk), (v, heads * dv), (beta, heads), (decay, heads * span)]
+    for tensor, width in outputs + ([(kq, kv_heads)] if kq is not None else []):
         _need(tensor.dtype == torch.float32 and tuple(tensor.shape) == (tokens, width) and tensor.is_contiguous(), "delta_prepare: bad output")
     ctx.lib.call(
         "b200_delta_prepare", ptr(proj), c_int(proj.stride(0)), ptr(decay_in), c_int(decay_in.stride(0)), ptr(taps),
         c_int(taps.shape[1]), ptr(conv_state), ptr(a_log), ptr(dt_bias), ptr(ctx.token_seq), ptr(ctx.seq_q_start),
         ptr(ctx.seq_q_len), ptr(ctx.seq_slot), c_int(tokens), c_int(ctx.num_seqs), c_int(heads), c_int(kv_heads), c_int(dk),
-        c_int(dv), ptr(q), ptr(k), ptr(v), ptr(beta), ptr(decay), c_int(dtype_code(proj.dtype)), ctx.stream,
+        c_int(dv), ptr(q), ptr(k), ptr(v), ptr(beta), ptr(decay), ptr(kq), c_int(dtype_code(proj.dtype)), ctx.stream,
     )
     ctx.lib.calls += 1  # the slot update is a launch of its own
 
@@ -852,15 +884,61 @@ def delta_recurrence(
 
 
 def delta_output(
-    ctx: StepContext, o: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, heads: int, dv: int, eps: float, out: torch.Tensor
+    ctx: StepContext, o: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, heads: int, dv: int, eps: float, out: torch.Tensor,
+    silu: bool = False,
 ) -> torch.Tensor:
+    """``o / rms(o) * weight * sigmoid(gate)`` per head; ``silu``: ``silu(gate)`` instead."""
     rows = o.shape[0]
     _need(o.dtype == torch.float32 and o.is_contiguous() and tuple(out.shape) == (rows, heads * dv) and out.is_contiguous(), "delta_output: bad operands")
     _need(gate.stride(1) == 1 and gate.shape[1] == heads * dv and gate.dtype == out.dtype, "delta_output: bad gate")
     _need(weight.dtype == torch.float32 and weight.numel() == dv, "delta_output: weight must be float32 [dv]")
     ctx.lib.call(
         "b200_delta_output", ptr(o), ptr(weight), ptr(gate), c_int(gate.stride(0)), c_int(rows), c_int(heads), c_int(dv),
-        c_float(eps), ptr(out), c_int(dtype_code(out.dtype)), ctx.stream,
+        c_float(eps), c_int(1 if silu else 0), ptr(out), c_int(dtype_code(out.dtype)), ctx.stream,
+    )
+    return out
+
+
+def delta_head_recurrence(
+    ctx: StepContext, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, beta: torch.Tensor, log_decay: torch.Tensor, kq: torch.Tensor,
+    state: torch.Tensor, out: torch.Tensor, heads: int, kv_heads: int, dk: int, dv: int,
+) -> torch.Tensor:
+    """The delta rule with one decay per head over every request's new tokens (operands as :func:`delta_prepare` leaves them)."""
+    tokens = q.shape[0]
+    _need(state.dtype == torch.float32 and tuple(state.shape[1:]) == (heads, dk, dv) and state.is_contiguous(), "delta_head_recurrence: the state is float32 [slots, heads, dk, dv]")
+    for tensor, width in ((q, kv_heads * dk), (k, kv_heads * dk), (v, heads * dv), (beta, heads), (log_decay, heads), (kq, kv_heads), (out, heads * dv)):
+        _need(tensor.dtype == torch.float32 and tuple(tensor.shape) == (tokens, width) and tensor.is_contiguous(), "delta_head_recurrence: bad operands")
+    ctx.lib.call(
+        "b200_delta_head_recurrence", ptr(q), ptr(k), ptr(v), ptr(beta), ptr(log_decay), ptr(kq), ptr(ctx.seq_q_start), ptr(ctx.seq_q_len),
+        ptr(ctx.seq_slot), c_int(ctx.num_seqs), c_int(ctx.max_q_len), c_int(heads), c_int(kv_heads), c_int(dk), c_int(dv), ptr(state), ptr(out), ctx.stream,
+    )
+    return out
+
+
+def delta_head_step_takes(ctx: StepContext, heads: int, kv_heads: int, dk: int, dv: int) -> bool:
+    """Whether the step is one of single tokens and the fused kernel takes the shape (``options["delta_step"] = "chain"``: never)."""
+    single = ctx.num_tokens == ctx.num_seqs == ctx.num_decode_seqs and ctx.options.get("delta_step", "auto") != "chain"
+    return single and bool(ctx.lib.lib.b200_delta_head_step_supported(heads, kv_heads, dk, dv))
+
+
+def delta_head_step(
+    ctx: StepContext, proj: torch.Tensor, taps: torch.Tensor, conv_state: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor,
+    norm_weight: torch.Tensor, eps: float, state: torch.Tensor, out: torch.Tensor, heads: int, kv_heads: int, dk: int, dv: int,
+) -> torch.Tensor:
+    """A step of single tokens in one kernel: ``proj`` rows are ``[q | k | v | b | a | gate]``; convolution, unit vectors, beta,
+    decay, recurrence, the output's norm and its silu gate. Moves ``conv_state`` and ``state`` on."""
+    channels = 2 * kv_heads * dk + heads * dv
+    _need(proj.is_contiguous() and proj.shape[0] == ctx.num_seqs and proj.shape[1] >= channels + 2 * heads + heads * dv, "delta_head_step: bad projections")
+    _need(taps.dtype == torch.float32 and taps.shape[0] == channels and taps.is_contiguous(), "delta_head_step: taps are float32 [channels, taps]")
+    _need(conv_state.dtype == proj.dtype and tuple(conv_state.shape[1:]) == (taps.shape[1] - 1, channels), "delta_head_step: bad convolution state")
+    _need(state.dtype == torch.float32 and tuple(state.shape[1:]) == (heads, dk, dv) and state.is_contiguous(), "delta_head_step: the state is float32 [slots, heads, dk, dv]")
+    for constant, count in ((a_log, heads), (dt_bias, heads), (norm_weight, dv)):
+        _need(constant.dtype == torch.float32 and constant.numel() == count, "delta_head_step: bad constants")
+    _need(tuple(out.shape) == (ctx.num_seqs, heads * dv) and out.is_contiguous() and out.dtype == proj.dtype, "delta_head_step: bad output")
+    ctx.lib.call(
+        "b200_delta_head_step", ptr(proj), c_int(proj.shape[1]), ptr(taps), c_int(taps.shape[1]), ptr(conv_state), ptr(a_log), ptr(dt_bias),
+        ptr(norm_weight), c_float(eps), ptr(ctx.seq_q_start), ptr(ctx.seq_slot), c_int(ctx.num_seqs), c_int(heads), c_int(kv_heads), c_int(dk),
+        c_int(dv), ptr(state), ptr(out), c_int(dtype_code(out.dtype)), ctx.stream,
     )
     return out
 

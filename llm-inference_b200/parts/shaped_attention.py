@@ -41,23 +41,25 @@ class ShapedAttention(Part):
     ``rel[bucket(distance), n]`` (``rel`` is ``[B, heads]``, see :func:`distance_buckets`); with ``chunk`` only keys of the
     query's own chunk of ``chunk`` positions (counted from the start of the request) are visible; with ``window`` only the
     last ``window`` keys, the query's own included, and the first ``keep_first`` of the request. Softmax over the
-    visible keys, or, with ``weights="sigmoid"``, each visible key weighs ``sigmoid(score + pb[n])`` and nothing is
+    visible keys, with ``sink`` with one more term ``exp(sink[n])`` in the denominator (no key, no value, not scaled), or, with ``weights="sigmoid"``, each visible key weighs ``sigmoid(score + pb[n])`` and nothing is
     normalised. With ``gate="head"`` head ``n``'s output is multiplied by ``sigmoid(W_g h)_n``. Then ``W_o`` (with ``v_bias`` and
     ``out_bias`` the values' and the output's product have biases too).
 
     The projections are one matrix ``[q | k | (v) | (g)]``; bias, norms, rotation and the cache write are one kernel.
     Keys and values share one arena row width (``padded_head_size``), as in the other mixers with ``dim`` and ``vdim``.
-    Tensor names: ``prefix + q | q.b | q.norm | k | k.b | k.norm | v | v.b | rel | pb | g | o | o.b``."""
+    Tensor names: ``prefix + q | q.b | q.norm | k | k.b | k.norm | v | v.b | rel | pb | sink | g | o | o.b``."""
 
     def __init__(self, *, prefix: str, hidden_size: int, heads: int, kv_heads: int, dim: int, vdim: int, scale: float, eps: float,
                  qk_norm: bool = True, qk_bias: bool = False, values: str = "projected", position: PartSpec | None = None,
                  softcap: float | None = None, distance_bias: dict | None = None, chunk: int = 0, gate: str | None = None,
                  window: int = 0, keep_first: int = 0, weights: str = "softmax", v_bias: bool = False, out_bias: bool = False,
-                 out_name: str = "branch") -> None:
+                 sink: bool = False, out_name: str = "branch") -> None:
         if heads % kv_heads:
             raise ValueError(f"{heads} query heads cannot share {kv_heads} kv heads")
         if weights not in ("softmax", "sigmoid"):
             raise ValueError(f"weights={weights!r} must be 'softmax' or 'sigmoid'")
+        if sink and weights != "softmax":
+            raise ValueError("a sink is a term of a softmax; sigmoid weights have none")
         if v_bias and values == "keys":
             raise ValueError("values that are the keys carry the keys' bias")
         if keep_first and not window:
@@ -75,7 +77,7 @@ class ShapedAttention(Part):
         self.softcap = float(softcap) if softcap else 0.0
         self.chunk = int(chunk or 0)
         self.window, self.keep_first, self.sigmoid = int(window or 0), int(keep_first or 0), weights == "sigmoid"
-        self.v_bias, self.has_out_bias = bool(v_bias), bool(out_bias)
+        self.v_bias, self.has_out_bias, self.has_sink = bool(v_bias), bool(out_bias), bool(sink)
         self.adds_out_bias = self.has_out_bias  # False: whoever takes the output adds `out_bias` (parts/parallel.py)
         self.out_bias: torch.Tensor | None = None
         # rows None: the table's row count is the checkpoint's (random weights need it named)
@@ -109,6 +111,8 @@ class ShapedAttention(Part):
                 specs.append(TensorSpec(p + "v.b", (self.kv_heads * self.vdim,)))
         if self.sigmoid:
             specs.append(TensorSpec(p + "pb", (self.heads,)))
+        if self.has_sink:
+            specs.append(TensorSpec(p + "sink", (self.heads,)))
         if self.has_bias:
             specs.append(TensorSpec(p + "rel", (self.bias_rows, self.heads)))
         if self.gate:
@@ -145,7 +149,8 @@ class ShapedAttention(Part):
             self.out_bias = get("o.b", f32).contiguous()
             self.out_bias_cast = self.out_bias.to(dtype)
         peak = self.bias_table.max(dim=1).values.contiguous() if self.bias_table is not None else None
-        self.shape = ops.ScoreShape(self.softcap, self.bias_table, self.chunk, peak, get("pb", f32).contiguous() if self.sigmoid else None)
+        self.shape = ops.ScoreShape(self.softcap, self.bias_table, self.chunk, peak, get("pb", f32).contiguous() if self.sigmoid else None,
+                                    get("sink", f32).contiguous() if self.has_sink else None)
         if self.position is not None:
             self.position.load(tensors, dtype, device)
 

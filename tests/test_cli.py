@@ -83,6 +83,7 @@ def test_replay_checks_its_options_and_needs_a_gpu(tmp_path):
     step = json.dumps({"step": 0, "entries": [{"id": "a", "tokens": [1, 2], "want": [1]}], "end": ["a"]}) + "\n"
     for extra, message in (
         (["--max-tokens", "0"], "--max-tokens must be positive"),
+        (["--max-tokens", "64", "--max-requests", "0"], "--max-requests must be positive"),
         (["--max-tokens", "64", "--page-size", "48"], "--page-size must divide 64"),
         (["--max-tokens", "64", "--dtype", "float16"], "invalid choice"),
     ):

@@ -145,12 +145,12 @@ def test_silu_mul(lib, dtype):
     torch.manual_seed(3)
     gate_up = (torch.randn(13, 2 * 272, device="cuda") * 4).to(dtype)
     out = torch.empty(13, 272, device="cuda", dtype=dtype)
-    ops.silu_mul(make_ctx(lib, positions=[0] * 13), gate_up, out)
+    ops.gated_mul(make_ctx(lib, positions=[0] * 13), gate_up, out)
     g, u = gate_up[:, 0::2].double(), gate_up[:, 1::2].double()  # gate and up interleaved
     torch.testing.assert_close(out.double(), g / (1 + torch.exp(-g)) * u, **tol(dtype))
     odd = (torch.randn(3, 2 * 37, device="cuda") * 4).to(dtype)  # not a multiple of eight
     out = torch.empty(3, 37, device="cuda", dtype=dtype)
-    ops.silu_mul(make_ctx(lib, positions=[0] * 3), odd, out)
+    ops.gated_mul(make_ctx(lib, positions=[0] * 3), odd, out)
     g, u = odd[:, 0::2].double(), odd[:, 1::2].double()
     torch.testing.assert_close(out.double(), g / (1 + torch.exp(-g)) * u, **tol(dtype))
 
@@ -190,7 +190,7 @@ def test_weight_streaming_gemm_matches_float64(lib, m, n, k, kernel):
     assert torch.equal(alone[0], out[m - 1])
     if n % 2 == 0:
         act = torch.full((m, n // 2), float("nan"), device="cuda", dtype=torch.bfloat16)
-        assert ops.linear_swiglu(ctx, x, w, act)
+        assert ops.linear_gated(ctx, x, w, act)
         g, u = want[:, 0::2], want[:, 1::2]
         torch.testing.assert_close(act.double(), g / (1 + torch.exp(-g)) * u, atol=2e-2, rtol=2e-2)
     assert int(ctx.err.item()) == 0
@@ -214,7 +214,7 @@ def test_tcgen05_gemm_takes_up_to_256_rows(lib, m, n, k):
     ops.linear(ctx, x, w, rounded)
     assert torch.equal(rounded, out.to(torch.bfloat16))  # the same sums, rounded once
     act = torch.full((m, n // 2), float("nan"), device="cuda", dtype=torch.bfloat16)
-    assert ops.linear_swiglu(ctx, x, w, act)
+    assert ops.linear_gated(ctx, x, w, act)
     want = x.double() @ w.double().T
     g, u = want[:, 0::2], want[:, 1::2]
     torch.testing.assert_close(act.double(), g / (1 + torch.exp(-g)) * u, atol=2e-2, rtol=2e-2)
@@ -322,11 +322,11 @@ def test_norm_folded_into_the_products_around_it(lib, kernel, m, hidden, inner, 
         error, floor = (out.double() - want).abs(), (chain.double() - want).abs()
         assert error.max() <= 1.5 * floor.max() + 1e-3 and error.mean() <= 1.2 * floor.mean() + 1e-4, (error.max(), floor.max())
     act = torch.full((m, wide // 2), float("nan"), device="cuda", dtype=torch.bfloat16)
-    assert ops.linear_swiglu(ctx, folded, w_out, act)
+    assert ops.linear_gated(ctx, folded, w_out, act)
     y = normed @ w_out.double().T
     gate, up = y[:, 0::2], y[:, 1::2]
     chain = torch.empty_like(act)
-    assert ops.linear_swiglu(ctx, h, w_out, chain)
+    assert ops.linear_gated(ctx, h, w_out, chain)
     want = gate / (1 + torch.exp(-gate)) * up
     error, floor = (act.double() - want).abs(), (chain.double() - want).abs()
     assert error.max() <= 1.5 * floor.max() + 1e-3 and error.mean() <= 1.2 * floor.mean() + 1e-4, (error.max(), floor.max())
