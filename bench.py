@@ -378,8 +378,25 @@ def dugalix_shape(width: int) -> dict:
             "layers": [first, attention, dict(first, mlp=mlp), attention][:DESIGN_LAYERS]}
 
 
-DESIGN_SHAPES = {"dugalix": dugalix_shape, "gunedra": gunedra_shape, "tunadra": tunadra_shape, "lerorax": lerorax_shape, "zetizen": zetizen_shape}
-CLOSEST = {"lerorax": "gunedra", "zetizen": "tunadra", "dugalix": "tunadra"}  # the existing design each is put beside by default (others: the Qwen2 shape)
+def tosipel_shape(width: int) -> dict:
+    """Layer sizes in the proportions of a real model of this design: attention heads of 128 sharing key/value heads as
+    the Qwen2 shape does, in windows of 1,024 positions; attention over latents of 512 numbers with queries out of a latent
+    of half the width; recurrent heads of 128 x 128 with four taps, pairs of heads sharing a q/k head; the dense
+    feed-forward of this width in every layer."""
+    heads, ff = DESIGN_SIZES[width]
+    mlp = {"kind": "dense", "ff": ff}
+    attention = {"type": "attention", "mlp": mlp, "mixer": {
+        "heads": heads, "kv_heads": heads // next(n for n in (6, 7, 5) if heads % n == 0), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 1024},
+        "rot": {"dims": 128, "base": 1e6}}}
+    latent = {"type": "latent_attention", "mlp": mlp, "mixer": {
+        "heads": heads, "dim": 128, "vdim": 128, "kv_rank": 512, "q_rank": width // 2, "scale": 128 ** -0.5}}
+    recurrent = {"type": "delta", "mlp": mlp, "mixer": {"heads": heads, "kv_heads": heads // 2, "dim": 128, "vdim": 128, "conv": 4}}
+    return {"architecture": "Tosipel", "vocab": DESIGN_VOCAB, "width": width, "embedding": {"scale": width ** 0.5}, "norm": {"eps": 1e-5},
+            "layers": [attention, latent, recurrent, attention][:DESIGN_LAYERS]}
+
+
+DESIGN_SHAPES = {"tosipel": tosipel_shape, "dugalix": dugalix_shape, "gunedra": gunedra_shape, "tunadra": tunadra_shape, "lerorax": lerorax_shape, "zetizen": zetizen_shape}
+CLOSEST = {"tosipel": "gunedra", "lerorax": "gunedra", "zetizen": "tunadra", "dugalix": "tunadra"}  # the existing design each is put beside by default (others: the Qwen2 shape)
 # The design each is put beside: the Qwen2 shape of equal width, or (--beside) another design's shape of equal width.
 
 
@@ -556,8 +573,9 @@ def main() -> int:
     parser.add_argument("--design-sizes", default="1536,3584", help="widths for --designs (1536, 3584 or 5120)")
     parser.add_argument("--design", choices=sorted(DESIGN_SHAPES), default="gunedra", help="which design --designs puts beside the Qwen2 shape")
     parser.add_argument("--beside", choices=["qwen2", "gunedra", "tunadra"], default=None,
-                        help="--designs: the shape of equal width to put the design beside (default: qwen2; for lerorax gunedra, the "
-                        "closest design: blocks that norm their branches' outputs, a delta rule, short convolutions, a dense feed-forward; for "
+                        help="--designs: the shape of equal width to put the design beside (default: qwen2; for lerorax and tosipel gunedra, the "
+                        "closest design: blocks that norm their branches' outputs, a delta rule, short convolutions, a dense feed-forward, "
+                        "and in tosipel as in gunedra attention over cached latents; for "
                         "zetizen and dugalix tunadra: attention mixers over the paged cache, a routed feed-forward with a shared expert, "
                         "and in tunadra as in dugalix a recurrent mixer with a matrix state)")
     args = parser.parse_args()

@@ -238,7 +238,7 @@ def bench_attention(args, decode: bool, mixed: bool = False) -> dict:
             continue
         bias = torch.randn(q_heads, args.bias_reach + 1, device="cuda") if args.bias_reach else None
         shape = ops.ScoreShape(args.softcap, bias, args.chunk, bias.max(dim=1).values.contiguous() if bias is not None else None,
-                               torch.zeros(q_heads, device="cuda") if args.sigmoid else None)
+                               torch.zeros(q_heads, device="cuda") if args.sigmoid else None, torch.zeros(q_heads, device="cuda") if args.sink else None)
         fns.append(lambda view=view, shape=shape: attention_dispatch.attend(ctx, view, q, out, q_heads, kv_heads, dim, dim**-0.5, shape=shape))
     # --rotate: back to back inside a CUDA graph, so that neither the host's launch cost nor
     # the idle gap before a lone launch enters (with one arena the cache stays in L2, as it
@@ -253,7 +253,7 @@ def bench_attention(args, decode: bool, mixed: bool = False) -> dict:
     if args.chunk and not mixed:
         flops = sum(4.0 * q_heads * dim * (p % args.chunk + 1) for p in positions)
     return {"kernel": ("mixed_" if mixed else "") + ("decode_attention" if decode else "prefill_attention"), "batch": len(lens), "context": args.context,
-            "tokens": len(positions), "softcap": args.softcap, "bias_reach": args.bias_reach, "chunk": args.chunk, "window": args.window, "keep_first": args.keep_first, "sigmoid": args.sigmoid, "loader": args.loader, "splits": args.splits, "stages": args.stages,
+            "tokens": len(positions), "softcap": args.softcap, "bias_reach": args.bias_reach, "chunk": args.chunk, "window": args.window, "keep_first": args.keep_first, "sigmoid": args.sigmoid, "sink": args.sink, "loader": args.loader, "splits": args.splits, "stages": args.stages,
             "layers": args.layers, "us": us, "GBps": kv_bytes / us / 1e3, "TFLOPs": flops / us / 1e6}
 
 
@@ -307,7 +307,8 @@ def bench_latent_attention(args, decode: bool) -> dict:
 def bench_delta_recurrence(args) -> dict:
     """The gated delta rule's recurrence (parts/delta_rule.py) over ``--batch`` requests of
     ``--tokens`` tokens each: ``--q-heads`` heads with states of ``--head-dim`` x ``--vdim``. Flops:
-    per token and head three products over the state (decay, k-dot and update, q-dot)."""
+    per token and head three products over the state (decay, k-dot and update, q-dot). ``--per-head``: the form with one
+    decay per head; ``--kv-heads`` q/k heads are shared by its heads."""
     from ..parts import ops
 
     heads, dk, dv, batch, tokens = args.q_heads, args.head_dim, args.vdim, args.batch, args.tokens
@@ -325,10 +326,39 @@ def bench_delta_recurrence(args) -> dict:
     decay = torch.rand(total, heads * dk, device="cuda") * 0.2 + 0.8
     state = torch.zeros(batch, heads, dk, dv, device="cuda")
     out = torch.empty(total, heads * dv, device="cuda")
-    us = time_launches(lambda: ops.delta_recurrence(ctx, q, k, v, beta, decay, state, out, heads, heads, dk, dv), args.iters)
     moved = 4.0 * (total * (3 * heads * dk + 2 * heads * dv + heads) + 2 * batch * heads * dk * dv)
-    return {"kernel": "delta_recurrence", "batch": batch, "tokens": tokens, "heads": heads, "dim": dk, "vdim": dv, "us": us,
+    run = lambda: ops.delta_recurrence(ctx, q, k, v, beta, decay, state, out, heads, heads, dk, dv)
+    if args.per_head:
+        kvh = args.kv_heads
+        q, k = (x.view(total, heads, dk)[:, :kvh].reshape(total, kvh * dk).contiguous() for x in (q, k))
+        kq = (q.view(total, kvh, dk) * k.view(total, kvh, dk)).sum(-1).contiguous()
+        decay = decay.view(total, heads, dk)[:, :, 0].log().contiguous()
+        moved = 4.0 * (total * (2 * kvh * dk + kvh + 2 * heads * dv + 2 * heads) + 2 * batch * heads * dk * dv)
+        run = lambda: ops.delta_head_recurrence(ctx, q, k, v, beta, decay, kq, state, out, heads, kvh, dk, dv)
+    us = time_launches(run, args.iters)
+    return {"kernel": "delta_head_recurrence" if args.per_head else "delta_recurrence", "batch": batch, "tokens": tokens, "heads": heads, "dim": dk, "vdim": dv, "us": us,
             "us_per_token": us / tokens, "GBps": moved / us / 1e3, "TFLOPs": 7.0 * total * heads * dk * dv / us / 1e6}
+
+
+def bench_delta_step(args) -> dict:
+    """Everything between the two products of the delta rule with one decay per head (parts/delta_rule.py, ``head_delta``) for one
+    token of each of ``--batch`` requests: the fused kernel, or with ``--plain`` the chain of kernels of prompt portions. Bytes: the
+    states and the convolution's history once each way, and the projections."""
+    from ..parts import PartSpec, build_part, ops
+
+    heads, kvh, dk, dv, batch, taps = args.q_heads, args.kv_heads, args.head_dim, args.vdim, args.batch, 4
+    ctx = make_ctx([5] * batch, list(range(batch)), [5] * batch, [1] * batch, {"delta_step": "chain" if args.plain else "auto"})
+    ctx.seq_slot = torch.arange(batch, dtype=torch.int32, device="cuda")
+    ctx.buffer = lambda name, shape, dtype=None, per_token=True: ctx.workspace.get(name, shape, dtype or torch.bfloat16, per_token=per_token)
+    part = build_part("mixer", PartSpec("head_delta", dict(prefix="", hidden_size=64, heads=heads, kv_heads=kvh, dim=dk, vdim=dv, taps=taps, eps=1e-5)))
+    part.load({s.name: torch.randn(s.shape) * 0.1 for s in part.tensor_specs()}, torch.bfloat16, torch.device("cuda"))
+    proj = torch.randn(batch, part.w_in.shape[0], device="cuda").to(torch.bfloat16)
+    state = torch.zeros(batch, heads, dk, dv, device="cuda")
+    history = torch.zeros(batch, taps - 1, part.channels, device="cuda", dtype=torch.bfloat16)
+    out = torch.empty(batch, heads * dv, device="cuda", dtype=torch.bfloat16)
+    us = time_launches(lambda: part.mix(ctx, proj, state, history, out), args.iters)
+    moved = 8.0 * batch * heads * dk * dv + 2.0 * (proj.numel() + out.numel() + 2 * history.numel())
+    return {"kernel": "delta_step", "batch": batch, "heads": heads, "kv_heads": kvh, "dim": dk, "vdim": dv, "chain": args.plain, "us": us, "GBps": moved / us / 1e3}
 
 
 def bench_wkv_recurrence(args) -> dict:
@@ -539,7 +569,7 @@ def bench_timeline(args) -> dict:
 def main(argv=None) -> int:
     parser = argparse.ArgumentParser(description=__doc__.split("\n\n")[0])
     parser.add_argument("kernel", choices=["gemm", "decode_attention", "prefill_attention", "resident", "timeline",
-                                           "latent_decode_attention", "latent_prefill_attention", "delta_recurrence", "wkv_recurrence",
+                                           "latent_decode_attention", "latent_prefill_attention", "delta_recurrence", "delta_step", "wkv_recurrence",
                                            "moe_experts", "mlstm", "delta_general_recurrence", "mixed_decode_attention",
                                            "mixed_prefill_attention"])
     parser.add_argument("--experts", type=int, default=32, help="moe_experts: number of experts")
@@ -570,6 +600,8 @@ def main(argv=None) -> int:
     parser.add_argument("--window", type=int, default=0)
     parser.add_argument("--keep-first", type=int, default=0, help="attention: first keys that stay visible in front of the window")
     parser.add_argument("--sigmoid", action="store_true", help="attention: sigmoid weights instead of a softmax")
+    parser.add_argument("--sink", action="store_true", help="attention: a sink per head in the softmax")
+    parser.add_argument("--per-head", action="store_true", help="delta_recurrence: the form with one decay per head")
     parser.add_argument("--plain", action="store_true")
     parser.add_argument("--softcap", type=float, default=0.0, help="attention: cap of the scores (0: none)")
     parser.add_argument("--bias-reach", type=int, default=0, help="attention: a random bias by distance up to this many positions (0: none)")
@@ -593,6 +625,8 @@ def main(argv=None) -> int:
         result = bench_latent_attention(args, args.kernel == "latent_decode_attention")
     elif args.kernel == "delta_recurrence":
         result = bench_delta_recurrence(args)
+    elif args.kernel == "delta_step":
+        result = bench_delta_step(args)
     elif args.kernel == "wkv_recurrence":
         result = bench_wkv_recurrence(args)
     elif args.kernel == "moe_experts":

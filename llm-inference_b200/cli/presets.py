@@ -92,7 +92,26 @@ def _dugalix(width, vocab, blocks, heads, kv_heads, experts, top, ff):
     return {"architecture": "Dugalix", "vocab": vocab, "width": width, "residual_mult": 0.5, "norm": {"eps": 1e-6}, "layers": layers}
 
 
+def _tosipel(width, vocab, blocks, heads, kv_heads, ff, shared=False):
+    """``blocks`` runs of (delta rule without a feed-forward, attention in a window, delta rule, attention over latents); with
+    ``shared`` a second run of all layers uses the first one's tensors."""
+    mlp = {"kind": "dense", "ff": ff}
+    delta = {"heads": heads, "kv_heads": heads // 2, "dim": 64, "vdim": 128, "conv": 4}
+    layers = [
+        {"type": "delta", "mlp": None, "mixer": delta},
+        {"type": "attention", "mlp": mlp, "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": 128, "vdim": 128, "scale": 0.1, "mask": {"size": 512},
+                                                    "rot": {"dims": 64, "base": 1e5}}},
+        {"type": "delta", "mlp": mlp, "mixer": delta},
+        {"type": "latent_attention", "mlp": mlp, "mixer": {"heads": heads, "dim": 96, "vdim": 128, "kv_rank": 256, "q_rank": 320, "scale": 96 ** -0.5}},
+    ] * blocks
+    if shared:
+        layers = layers + [dict(layer, weights_of=index) for index, layer in enumerate(layers)]
+    return {"architecture": "Tosipel", "vocab": vocab, "width": width, "embedding": {"scale": float(width) ** 0.5}, "norm": {"eps": 1e-5}, "layers": layers}
+
+
 PRESETS = {
+    "tosipel-small": _tosipel(512, 8192, 1, 8, 2, 1024, shared=True),
+    "tosipel-1b": _tosipel(2048, 32768, 4, 16, 4, 5632),
     "dugalix-small": _dugalix(512, 8192, 2, 8, 2, 16, 2, 256),
     "dugalix-1b": _dugalix(2048, 32768, 6, 16, 4, 16, 2, 512),
     "zetizen-small": _zetizen(512, 8192, 2, 8, 2, 16, 2, 256),

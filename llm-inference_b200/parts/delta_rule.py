@@ -161,10 +161,13 @@ class HeadDeltaRule(Part):
         return sum(w.numel() * w.element_size() for w in (self.w_in, self.w_o))
 
     def forward(self, ctx: StepContext, cache: CacheView, h: torch.Tensor) -> torch.Tensor:
+        proj = ops.linear(ctx, h, self.w_in, ctx.buffer("delta_in", (ctx.num_tokens, self.w_in.shape[0])))
+        y = self.mix(ctx, proj, *cache.state, ctx.buffer("attn", (ctx.num_tokens, self.heads * self.vdim)))
+        return ops.linear(ctx, y, self.w_o, ctx.buffer(self.out_name, (ctx.num_tokens, self.hidden_size)))
+
+    def mix(self, ctx: StepContext, proj: torch.Tensor, state: torch.Tensor, conv_state: torch.Tensor, y: torch.Tensor) -> torch.Tensor:
+        """Everything between the two products."""
         t, heads, kvh, dk, dv = ctx.num_tokens, self.heads, self.kv_heads, self.dim, self.vdim
-        state, conv_state = cache.state
-        proj = ops.linear(ctx, h, self.w_in, ctx.buffer("delta_in", (t, self.w_in.shape[0])))
-        y = ctx.buffer("attn", (t, heads * dv))
         if ops.delta_head_step_takes(ctx, heads, kvh, dk, dv):
             ops.delta_head_step(ctx, proj, self.taps_w, conv_state, self.a_log, self.dt_bias, self.norm_weight, self.eps, state, y, heads, kvh, dk, dv)
         else:
@@ -176,7 +179,7 @@ class HeadDeltaRule(Part):
                               q, k, v, beta, decay, kq)
             o = ops.delta_head_recurrence(ctx, q, k, v, beta, decay, kq, state, ctx.buffer("delta_o", (t, heads * dv), f32), heads, kvh, dk, dv)
             ops.delta_output(ctx, o, self.norm_weight, proj[:, a_at + heads :], heads, dv, self.eps, y, silu=True)
-        return ops.linear(ctx, y, self.w_o, ctx.buffer(self.out_name, (t, self.hidden_size)))
+        return y
 
 
 class GeneralDeltaRule(Part):

@@ -207,3 +207,14 @@ def forward(config: dict, weights: dict, tokens, state: dict | None = None, laye
         if layer_outputs is not None:
             layer_outputs.append(x.copy())
     return linear(offset_norm(x, w["final.norm"], eps), w["head"])
+
+
+def greedy(config: dict, weights: dict, prompt, count: int) -> list[int]:
+    """``count`` tokens, each the likeliest after everything in front of it."""
+    state: dict = {}
+    logits = forward(config, weights, prompt, state)[-1]
+    out: list[int] = []
+    while len(out) < count:
+        out.append(int(np.argmax(logits)))
+        logits = forward(config, weights, [out[-1]], state)[-1]
+    return out

@@ -132,9 +132,10 @@ def test_blend_with_the_previous_token_across_steps_and_slots(name, hidden):
 PORTIONS = (7, 1, 2, 9, 1, 1, 1, 16, 1, 1, 1, 1, 28)  # 70 tokens; single ones at 7, 19 to 21 and 38 to 41: both sides of page edges
 
 
-def run_in_portions(mixer, weights, dtype, inputs, total, poison=True):
+def run_in_portions(mixer, weights, dtype, inputs, total, options=None):
     """Request 10 in PORTIONS beside request 11 (three tokens, then one by one), pages of 8 and slots full of NaN."""
     runner, cache, _ = context_for({0: mixer.cache_spec()}, dtype, [1])
+    runner.options.update(options or {})
     for group in cache.groups:
         group.arena.fill_(float("nan"))  # pages are not cleared between requests: a request reads only what it wrote
     for arrays in cache.states.values():
