@@ -308,14 +308,14 @@ def bench_delta_recurrence(args) -> dict:
     """The gated delta rule's recurrence (parts/delta_rule.py) over ``--batch`` requests of
     ``--tokens`` tokens each: ``--q-heads`` heads with states of ``--head-dim`` x ``--vdim``. Flops:
     per token and head three products over the state (decay, k-dot and update, q-dot). ``--per-head``: the form with one
-    decay per head; ``--kv-heads`` q/k heads are shared by its heads."""
+    decay per head; ``--kv-heads`` q/k heads are shared by its heads; ``--portions``: chunk by chunk or token by token."""
     from ..parts import ops
 
     heads, dk, dv, batch, tokens = args.q_heads, args.head_dim, args.vdim, args.batch, args.tokens
     runs, starts = [tokens] * batch, [0] * batch
     positions = [p for r in runs for p in range(r)]
     token_seq = [i for i, r in enumerate(runs) for _ in range(r)]
-    ctx = make_ctx(positions, token_seq, starts, runs)
+    ctx = make_ctx(positions, token_seq, starts, runs, {"delta_portions": args.portions})
     ctx.seq_slot = torch.arange(batch, dtype=torch.int32, device="cuda")
     total = batch * tokens
     unit = lambda x: x / x.norm(dim=-1, keepdim=True)
@@ -602,6 +602,7 @@ def main(argv=None) -> int:
     parser.add_argument("--sigmoid", action="store_true", help="attention: sigmoid weights instead of a softmax")
     parser.add_argument("--sink", action="store_true", help="attention: a sink per head in the softmax")
     parser.add_argument("--per-head", action="store_true", help="delta_recurrence: the form with one decay per head")
+    parser.add_argument("--portions", default="auto", choices=["auto", "chunks", "tokens"], help="delta_recurrence --per-head: how portions are walked")
     parser.add_argument("--plain", action="store_true")
     parser.add_argument("--softcap", type=float, default=0.0, help="attention: cap of the scores (0: none)")
     parser.add_argument("--bias-reach", type=int, default=0, help="attention: a random bias by distance up to this many positions (0: none)")

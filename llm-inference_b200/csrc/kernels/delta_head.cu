@@ -164,7 +164,7 @@ constexpr int kStepWarps = kStepThreads / 32;
 // A warp holds 32 neighbouring columns of `slice_rows` rows of S, a row's 32 numbers in one access. The heads that share a
 // q/k head are one thread-block cluster (its first block moves their convolution history on, once all have read it).
 template <typename T, int PER>
-__global__ void __launch_bounds__(kStepThreads, 1)
+__global__ void __launch_bounds__(kStepThreads, PER <= 32 ? 2 : 1)
 delta_head_step_kernel(const T* proj, const float* __restrict__ taps_w, T* conv_state, const float* __restrict__ a_log,
                        const float* __restrict__ dt_bias, const float* __restrict__ norm_weight, const int* __restrict__ seq_q_start,
                        const int* __restrict__ seq_slot, const StepShape p, float* state, T* out) {

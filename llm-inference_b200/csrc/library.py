@@ -91,6 +91,7 @@ _SIGNATURES: dict[str, list] = {
     "b200_delta_recurrence": [c_void_p] * 8 + [c_int] * 5 + [c_void_p] * 3,
     "b200_delta_output": [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_int, c_void_p, c_int, c_void_p],
     "b200_delta_head_recurrence": [c_void_p] * 9 + [c_int] * 6 + [c_void_p] * 3,
+    "b200_delta_chunks": [c_void_p] * 8 + [c_int] * 6 + [c_void_p] * 6,
     "b200_delta_head_step": [c_void_p, c_int, c_void_p, c_int] + [c_void_p] * 4 + [c_float, c_void_p, c_void_p] + [c_int] * 5
                             + [c_void_p, c_void_p, c_int, c_void_p],
     "b200_embedding_sinusoid": [c_void_p] * 4 + [c_float, c_void_p, c_int, c_int, c_int, c_int, c_int, c_void_p, c_void_p],
@@ -165,6 +166,8 @@ class KernelLibrary:
         self.lib.b200_latent_attention_mma_supported.restype = c_int
         self.lib.b200_latent_attention_mma_scratch.argtypes = [c_int] * 5
         self.lib.b200_latent_attention_mma_scratch.restype = c_int64
+        self.lib.b200_delta_chunks_supported.argtypes = [c_int] * 4
+        self.lib.b200_delta_chunks_supported.restype = c_int
         self.lib.b200_delta_head_step_supported.argtypes = [c_int] * 4
         self.lib.b200_delta_head_step_supported.restype = c_int
         self.lib.b200_moe_tile_rows.argtypes = []

@@ -899,15 +899,31 @@ def delta_output(
     return out
 
 
+DELTA_CHUNK_FROM = 64  # longest portion that is walked token by token: two more launches and a whole chunk a block cost about as much
+
+
 def delta_head_recurrence(
     ctx: StepContext, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, beta: torch.Tensor, log_decay: torch.Tensor, kq: torch.Tensor,
     state: torch.Tensor, out: torch.Tensor, heads: int, kv_heads: int, dk: int, dv: int,
 ) -> torch.Tensor:
-    """The delta rule with one decay per head over every request's new tokens (operands as :func:`delta_prepare` leaves them)."""
+    """The delta rule with one decay per head over every request's new tokens (operands as :func:`delta_prepare` leaves them).
+    Portions of more than ``DELTA_CHUNK_FROM`` tokens run chunk by chunk (two kernels, the 32 x 32 matrices of all chunks in
+    between), shorter ones token by token; ``options["delta_portions"]``: ``"chunks"`` or ``"tokens"`` forces one of them."""
     tokens = q.shape[0]
     _need(state.dtype == torch.float32 and tuple(state.shape[1:]) == (heads, dk, dv) and state.is_contiguous(), "delta_head_recurrence: the state is float32 [slots, heads, dk, dv]")
     for tensor, width in ((q, kv_heads * dk), (k, kv_heads * dk), (v, heads * dv), (beta, heads), (log_decay, heads), (kq, kv_heads), (out, heads * dv)):
         _need(tensor.dtype == torch.float32 and tuple(tensor.shape) == (tokens, width) and tensor.is_contiguous(), "delta_head_recurrence: bad operands")
+    choice = ctx.options.get("delta_portions", "auto")
+    if choice == "chunks" or (choice == "auto" and ctx.max_q_len > DELTA_CHUNK_FROM and ctx.lib.lib.b200_delta_chunks_supported(heads, kv_heads, dk, dv)):
+        attn, solve = (ctx.buffer("delta_" + name, (tokens, heads * 32), torch.float32) for name in ("chunk_attn", "chunk_solve"))
+        factors = ctx.buffer("delta_chunk_factors", (tokens, heads * 2), torch.float32)
+        ctx.lib.call(
+            "b200_delta_chunks", ptr(q), ptr(k), ptr(v), ptr(beta), ptr(log_decay), ptr(ctx.seq_q_start), ptr(ctx.seq_q_len), ptr(ctx.seq_slot),
+            c_int(ctx.num_seqs), c_int(ctx.max_q_len), c_int(heads), c_int(kv_heads), c_int(dk), c_int(dv), ptr(attn), ptr(solve), ptr(factors),
+            ptr(state), ptr(out), ctx.stream,
+        )
+        ctx.lib.calls += 1  # two kernels
+        return out
     ctx.lib.call(
         "b200_delta_head_recurrence", ptr(q), ptr(k), ptr(v), ptr(beta), ptr(log_decay), ptr(kq), ptr(ctx.seq_q_start), ptr(ctx.seq_q_len),
         ptr(ctx.seq_slot), c_int(ctx.num_seqs), c_int(ctx.max_q_len), c_int(heads), c_int(kv_heads), c_int(dk), c_int(dv), ptr(state), ptr(out), ctx.stream,

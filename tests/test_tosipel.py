@@ -321,10 +321,10 @@ DELTA = {
 
 @pytest.mark.parametrize("name", ["float32", "bfloat16"])
 @pytest.mark.parametrize("case", sorted(DELTA))
-@pytest.mark.parametrize("step", ["auto", "chain"])
+@pytest.mark.parametrize("step", ["auto", "tokens", "chunks"])
 def test_delta_rule_alone_in_portions_beside_another_request(name, case, step):
     """70 tokens in portions beside another request, slots full of NaN before; steps in which both feed one token run the fused
-    kernel ("chain": the kernels of prompt portions in every step). The test asserts that a lost state, a lost convolution
+    kernel ("tokens", "chunks": the kernels of prompt portions in every step, token by token or 32 tokens at a time). The test asserts that a lost state, a lost convolution
     history, a missing decay, a read-out of the old state and unit vectors left out would show."""
     dtype, hidden, total = DTYPES[name], 48, 70
     layer = DELTA[case]
@@ -349,16 +349,21 @@ def test_delta_rule_alone_in_portions_beside_another_request(name, case, step):
     finally:
         plain.delta_step = original
     mixer.load(weights, dtype, torch.device(DEVICE))  # the history is kept in the weights' dtype
-    got = run_in_portions(mixer, weights, dtype, inputs, total, {"delta_step": step})
+    if step == "chunks" and m["dim"] > 256:
+        pytest.skip("chunks take up to 256 key channels")
+    options = {} if step == "auto" else {"delta_step": "chain", "delta_portions": step}
+    got = run_in_portions(mixer, weights, dtype, inputs, total, options)
     np.testing.assert_allclose(got[10], want[10], **CLOSE[name])
     np.testing.assert_allclose(got[11], want[11], **CLOSE[name])
 
 
 @pytest.mark.parametrize("name", ["float32", "bfloat16"])
-@pytest.mark.parametrize("case", ["three kv heads", "whole warps", "odd", "eight heads on one"])
-def test_delta_rule_long_portions_and_many_single_tokens(name, case):
-    """500 tokens: as one portion beside others of 1 to 129 tokens, then the same as 60 single tokens behind a portion; heads
-    that keep hundreds of tokens and heads that forget in a few."""
+@pytest.mark.parametrize("case", ["three kv heads", "whole warps", "odd", "eight heads on one", "nine heads on one", "wide values"])
+@pytest.mark.parametrize("portions", ["auto", "tokens"])
+def test_delta_rule_long_portions_and_many_single_tokens(name, case, portions):
+    """500 tokens: as one portion beside others of 1 to 129 tokens, then the same as 60 single tokens behind a portion, then cut
+    around multiples of 32 (the chunks of the kernels that take 32 tokens at a time start with a portion); heads that keep hundreds
+    of tokens and heads that forget in a few."""
     from llm_inference_b200.cache import PagedCache
     from llm_inference_b200.engine.runner import ModelRunner
 
@@ -375,7 +380,7 @@ def test_delta_rule_long_portions_and_many_single_tokens(name, case):
         cache = PagedCache({0: mixer.cache_spec()}, dtype=dtype, device=device, page_size=8, max_num_sequences=6, max_model_length=512, step_tokens=1024, num_pages=8)
         for array in cache.states[0]:
             array.fill_(float("nan"))
-        runner = ModelRunner(SimpleNamespace(device=device, dtype=dtype), cache, max_batch_tokens=1024)
+        runner = ModelRunner(SimpleNamespace(device=device, dtype=dtype), cache, max_batch_tokens=1024, options={"delta_portions": portions})
         for rid in lengths:
             cache.open(rid)
         at, parts = 0, []
@@ -393,6 +398,44 @@ def test_delta_rule_long_portions_and_many_single_tokens(name, case):
         runner.check()
         assert at == total
         np.testing.assert_allclose(np.concatenate(parts), want[10], **CLOSE[name])
+
+
+def test_chunks_with_decays_that_end_a_memory_at_once_and_keys_that_repeat():
+    """float32, the recurrences' kernels on given operands: log decays of zero, tiny ones, and down to -400 in the middle of a chunk;
+    keys that repeat token after token with beta near one (the triangular system at its stiffest); 32 tokens at a time, token by
+    token and the 64-bit recurrence agree, and a state that comes in counts."""
+    from llm_inference_b200.parts import StateSpec, ops
+
+    heads, kvh, dk, dv, n = 4, 2, 40, 28, 150
+    rng = np.random.default_rng(3)
+    unit = lambda x: x / np.linalg.norm(x, axis=-1, keepdims=True)
+    k, q = unit(rng.normal(size=(n, kvh, dk))), unit(rng.normal(size=(n, kvh, dk)))
+    k[20:60] = k[20]
+    v, beta = rng.normal(size=(n, heads, dv)), rng.uniform(0.95, 1.0, (n, heads))
+    log_decay = -np.exp(rng.normal(-5, 2, (n, heads)))
+    log_decay[:, 1] = 0.0
+    log_decay[[17, 40, 41, 97], 2] = [-400.0, -90.0, -400.0, -30.0]
+    start = rng.normal(size=(heads, dk, dv))
+    q, k, v, beta, log_decay, start = (a.astype(np.float32) for a in (q, k, v, beta, log_decay, start))
+    S = start.astype(np.float64)
+    want = np.zeros((n, heads, dv))
+    for t in range(n):
+        for h in range(heads):
+            S[h], want[t, h] = plain.delta_step(S[h], q[t, h // 2].astype(np.float64), k[t, h // 2].astype(np.float64), v[t, h].astype(np.float64),
+                                                np.exp(float(log_decay[t, h])), float(beta[t, h]))
+    device = [torch.from_numpy(np.ascontiguousarray(a.reshape(n, -1))).cuda() for a in (q, k, v, beta, log_decay, (q * k).sum(-1))]
+    for choice in ("tokens", "chunks"):
+        runner, cache, ctx = context_for({0: StateSpec(((heads, dk, dv),), (torch.float32,))}, torch.float32, [2])
+        ctx.options = {"delta_portions": choice}
+        state = cache.states[0][0]
+        state[:] = torch.from_numpy(start).cuda()
+        ctx.num_tokens, ctx.num_seqs, ctx.max_q_len = n, 1, n
+        ctx.seq_q_start, ctx.seq_q_len = (torch.tensor([x], dtype=torch.int32, device="cuda") for x in (0, n))
+        out = torch.full((n, heads * dv), float("nan"), device="cuda")
+        ops.delta_head_recurrence(ctx, *device, state, out, heads, kvh, dk, dv)
+        runner.check()
+        np.testing.assert_allclose(as64(out).reshape(want.shape), want, atol=2e-5, rtol=2e-5, err_msg=choice)
+        np.testing.assert_allclose(as64(state[int(ctx.seq_slot[0])]), S, atol=2e-5, rtol=2e-5, err_msg=choice)
 
 
 # --- the gated unit ----------------------------------------------------------------------------------------------------------
